@@ -19,7 +19,7 @@ CC_MAX_DIMS = 4
 F32, F16, Q4_0, Q4_1, Q5_0, Q5_1, Q8_0, Q8_1 = 0, 1, 2, 3, 6, 7, 8, 9
 Q2_K, Q3_K, Q4_K, Q5_K, Q6_K, Q8_K = 10, 11, 12, 13, 14, 15
 I32, BF16 = 26, 30
-ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_SWISH, ACT_SIGMOID = 0, 1, 2, 3, 4
+ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_SWISH, ACT_SIGMOID, ACT_RELU_SQUARED = 0, 1, 2, 3, 4, 5
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
 ROPE_LLAMA, ROPE_NEOX = 0, 1
 QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_ROW = 0, 1, 2
@@ -141,8 +141,26 @@ class clr_layer_weights(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in CLR_WEIGHT_FIELDS]
 
 
+class cpr_layer_config(C.Structure):            # include/crabml_papunex.h
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "kv_from")] + [("scale", C.c_float), ("rot_mag", C.c_float)] + \
+               [(n, C.c_int32) for n in ("s_heads", "s_vdim", "s_state", "s_groups", "s_conv", "s_norm_groups", "ff_kind", "ff", "experts", "top", "shared")] + \
+               [("route_scale", C.c_float)]
+
+
+class cpr_config(C.Structure):
+    _fields_ = [("n_layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("norm_eps", C.c_float), ("softcap", C.c_float), ("chunk", C.c_int32), ("max_seq", C.c_int32)]
+
+
+CPR_WEIGHT_FIELDS = ("norm1", "norm2", "h_stack", "dkv_norm", "uk", "uv", "uk_t", "uv_f32", "sink", "rot_freq", "o", "in", "conv", "conv_bias", "dt_bias", "a_log", "d_skip",
+                     "s_norm", "s_o", "up", "down", "router", "shared_gate")
+
+
+class cpr_layer_weights(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in CPR_WEIGHT_FIELDS]
+
+
 class cc_route_params(C.Structure):              # include/crabml_seqops.h
-    _fields_ = [(n, C.c_int32) for n in ("score", "top", "n_groups", "keep_groups", "group_top", "renormalise")] + [("renorm_eps", C.c_float)]
+    _fields_ = [(n, C.c_int32) for n in ("score", "top", "n_groups", "keep_groups", "group_top", "renormalise")] + [("renorm_eps", C.c_float), ("scale", C.c_float)]
 
 
 class cc_glu_params(C.Structure):
@@ -283,6 +301,16 @@ def load_library(build_if_missing: bool = True):
         "cc_masked_attention_capped": (i32, [vp, pv, pv, pv, i64, i32, i32, i32, i32, i32, i32, f32, f32, pv, pp]),
         "cc_retention": (i32, [vp, pv, pv, pv, pv, f32, pv, i32, i32, i32, pp]),
         "cc_gated_diagonal_recurrence": (i32, [vp, pv, pv, pv, pv, f32, i32, pv, pv, i32, pv, pp]),
+        "cc_activate_inplace": (i32, [vp, pv, i32]),
+        "cc_softcap_inplace": (i32, [vp, pv, f32]),
+        "cc_short_conv_cols": (i32, [vp, pv, i32, pv, pv, pv, i32, pp]),
+        "cc_state_space_scan_cols": (i32, [vp, pv, pv, i32, pv, pv, pv, pv, i32, i32, i32, i32, pp]),
+        "cc_head_project_gated": (i32, [vp, pv, pv, i32, pv, i32, pp]),
+        "cc_latent_query_append": (i32, [vp, pv, i32, pv, i32, i32, pv, f32, i64, pv, i32, pv, pv, f32, pp]),
+        "cc_moe_route_shared": (i32, [vp, pv, pv, pv, pv, i32, C.POINTER(cc_route_params), pp, pp]),
+        "cc_moe_experts_act": (i32, [vp, pv, pv, pv, pv, pv, i32, i32, i32, pp]),
+        "cc_feed_forward_act": (i32, [vp, pv, pv, pv, i32, pp]),
+        "cpr_runner_create": (i32, [vp, C.POINTER(cpr_config), C.POINTER(cpr_layer_config), C.POINTER(cpr_layer_weights), vp, vp, vp, pp]),
         "clr_runner_create": (i32, [vp, C.POINTER(clr_config), C.POINTER(clr_layer_config), C.POINTER(clr_layer_weights), vp, vp, vp, vp, vp, pp]),
         "cvr_runner_create": (i32, [vp, C.POINTER(cvr_config), C.POINTER(cvr_layer_config), C.POINTER(cvr_layer_weights), vp, vp, vp, vp, pp]),
         "csr_runner_destroy": (None, [vp]),

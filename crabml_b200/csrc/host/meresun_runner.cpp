@@ -14,7 +14,7 @@
 #include <vector>
 
 #include "../../../include/crabml_meresun.h"
-#include "seq_runner.hpp"
+#include "mixers.hpp"
 
 using crabml::CudaTensor;
 using crabml::TensorError;
@@ -23,8 +23,8 @@ namespace {
 
 struct Layer {
     cmr_layer_config c{};
-    CudaTensor norm1, h_stack, dq_norm, uq, dkv_norm, uk, uv, uk_t, uv_f32, sink, rot_freq, o, rg1_b, rg2_b, down, act, router, correction, e_gate, e_up, e_down, side_table,
-        side_gate, side_proj, side_norm;
+    CudaTensor norm1, h_stack, dq_norm, uq, o, rg1_b, rg2_b, down, act, router, correction, e_gate, e_up, e_down, side_table, side_gate, side_proj, side_norm;
+    crabml::LatentAttention att;
     std::vector<int32_t> widths;                         // column blocks of h_stack's product, in order
     int i_g1 = -1, i_g2 = -1, i_up = -1;                 // which block is which (blocks 0 and 1: the cache row, the query latent); -1: absent
     int64_t ring = 0;            // rows of the latent cache of one run of this layer
@@ -37,11 +37,7 @@ struct Run {
 struct State : crabml::SeqState {
     std::vector<CudaTensor> ring;          // per run: [rows, kv_rank + rot_dim]
 };
-const cc_view* opt(const CudaTensor& t, cc_view& store) {
-    if (!t.valid()) return nullptr;
-    store = t.view();
-    return &store;
-}
+using crabml::opt_view;
 
 struct Runner : csr_runner {
     cmr_config conf{};
@@ -69,56 +65,10 @@ struct Runner : csr_runner {
 
     // ckv: the new tokens' raw cache rows W_dkv h; cq: their raw query latents W_dq h
     CudaTensor mixer(const Layer& L, CudaTensor& ring, const CudaTensor& ckv, CudaTensor cq, int64_t pos0) {
-        const auto& c = L.c;
-        const int64_t n = ckv.shape()[0];
-        if (c.window <= 0 && pos0 + n > L.ring) throw TensorError("a sequence of " + std::to_string(pos0 + n) + " tokens does not fit the cache of " + std::to_string(L.ring));
-        cc_view fq{};
-        const cc_view* freq = opt(L.rot_freq, fq);
-        // the cache row of every new token
-        {
-            cc_view rv = ring.view(), cv = ckv.view(), nw{};
-            check(cc_latent_ring_append(dev, &rv, &cv, opt(L.dkv_norm, nw), conf.norm_eps, c.kv_rank, freq, c.rot_mag, pos0));
-        }
-        // queries through their latent
-        cq = norm(cq, L.dq_norm, 1);
-        CudaTensor q = L.uq.matmul_vec(cq);
-        cc_view qv = q.view();
-        cc_buf* b = nullptr;
-        cc_view rv = ring.view(), sk{};
-        CudaTensor o;
-        if (n * c.heads > 64) {
-            if (freq) check(cc_rope_pairs(dev, &qv, c.heads, c.dim + c.rot_dim, c.dim, freq, c.rot_mag, pos0));
-            // many rows: expand the cached rows once for all queries of the pass.  The expansion keeps the ring's row order (position p in
-            // row p % ring), so the attention reads it like the ring itself; rows no token has written yet are never visible.
-            const int64_t rows = std::min<int64_t>(L.ring, pos0 + n);
-            const int64_t cols = (int64_t)c.kv_rank + c.rot_dim;
-            CudaTensor lat = CudaTensor(ring).with_strider(crabml::TensorStrider({rows, c.kv_rank}, {cols, 1})).contiguous();
-            CudaTensor kp = L.uk.matmul_vec(lat), v = L.uv.matmul_vec(lat);
-            cc_view kpv = kp.view(), vv = v.view();
-            check(cc_head_concat_shared(dev, &kpv, &rv, c.heads, c.kv_rank, c.rot_dim, &b));
-            CudaTensor keys = adopt(b, {rows, (int64_t)c.heads * (c.dim + c.rot_dim)});
-            cc_view kv = keys.view();
-            b = nullptr;
-            check(cc_window_attention_sink(dev, &qv, nullptr, 0.0f, &kv, &vv, pos0, c.heads, c.heads, c.dim + c.rot_dim, c.vdim, c.window, c.scale, nullptr, nullptr,
-                                           opt(L.sink, sk), &b));
-            o = adopt(b, {n, (int64_t)c.heads * c.vdim});
-        } else {
-            // few rows: all heads read the one cached row per position; keys are whole rows, values their first kv_rank columns.  The
-            // query's rotated part is turned while it is carried past the fold.
-            cc_view ukv = L.uk_t.view();
-            check(cc_head_project(dev, &qv, &ukv, c.heads, c.rot_dim, freq, c.rot_mag, pos0, &b));
-            CudaTensor ql = adopt(b, {n, (int64_t)c.heads * (c.kv_rank + c.rot_dim)});
-            cc_view qlv = ql.view();
-            b = nullptr;
-            check(cc_window_attention_sink(dev, &qlv, nullptr, 0.0f, &rv, nullptr, pos0, c.heads, 1, c.kv_rank + c.rot_dim, c.kv_rank, c.window, c.scale, nullptr, nullptr,
-                                           opt(L.sink, sk), &b));
-            CudaTensor ol = adopt(b, {n, (int64_t)c.heads * c.kv_rank});
-            cc_view olv = ol.view(), uvv = L.uv_f32.view();
-            b = nullptr;
-            check(cc_head_project(dev, &olv, &uvv, c.heads, 0, nullptr, 1.0f, 0, &b));
-            o = adopt(b, {n, (int64_t)c.heads * c.vdim});
-        }
-        return L.o.matmul_vec(o);
+        CudaTensor q = L.uq.matmul_vec(norm(cq, L.dq_norm, 1));                       // queries through their latent
+        if (L.att.few_rows(ckv.shape()[0])) return L.o.matmul_vec(L.att.attend_few(*this, ring, q, 0, &ckv, 0, nullptr, 0, pos0));
+        L.att.append(*this, ring, ckv, pos0);
+        return L.o.matmul_vec(L.att.attend_many(*this, ring, q, pos0));
     }
 
     // z: the dense feed-forward's W_up h (unused by a routed one)
@@ -133,7 +83,7 @@ struct Runner : csr_runner {
         cc_view hv = h.view(), rw = L.router.view(), cv{};
         cc_buf *ids = nullptr, *wts = nullptr, *ob = nullptr;
         const cc_route_params rp = {CC_ROUTE_SIGMOID, c.top, c.groups, c.keep_groups, 2, 1, 1e-20f};
-        check(cc_moe_route_ex(dev, &hv, &rw, opt(L.correction, cv), &rp, &ids, &wts));
+        check(cc_moe_route_ex(dev, &hv, &rw, opt_view(L.correction, cv), &rp, &ids, &wts));
         CudaTensor tid = adopt(ids, {n, c.top}), tw = adopt(wts, {n, c.top});
         cc_view iv = tid.view(), wv = tw.view(), g = L.e_gate.view(), u = L.e_up.view(), d = L.e_down.view();
         const cc_glu_params glu = {CC_ACT_SWISH, 1.702f, c.limit, 1.0f};
@@ -161,14 +111,7 @@ struct Runner : csr_runner {
             }
             {
                 CudaTensor h = norm(x, L.norm1, conf.norm_groups);
-                std::vector<CudaTensor> part;
-                {
-                    CudaTensor all = L.h_stack.matmul_vec(h);
-                    cc_view av = all.view();
-                    std::vector<cc_buf*> outs(L.widths.size(), nullptr);
-                    check(cc_split_cols(dev, &av, (int32_t)L.widths.size(), L.widths.data(), outs.data()));
-                    for (size_t p = 0; p < outs.size(); p++) part.push_back(adopt(outs[p], {n, L.widths[p]}));
-                }
+                std::vector<CudaTensor> part = crabml::split_columns(*this, L.h_stack.matmul_vec(h), L.widths);
                 CudaTensor y = mixer(L, s.ring[ri], part[0], part[1], pos0);
                 CudaTensor g1, f, g2;
                 if (L.i_g1 >= 0) g1 = part[L.i_g1];
@@ -177,7 +120,7 @@ struct Runner : csr_runner {
                     if (L.i_g2 >= 0) g2 = part[L.i_g2];
                 }
                 cc_view xv = x.view(), yv = y.view(), g1v{}, b1v{}, fv{}, g2v{}, b2v{};
-                check(cc_gated_sum(dev, &xv, 1, &yv, opt(g1, g1v), opt(L.rg1_b, b1v), opt(f, fv), opt(g2, g2v), opt(L.rg2_b, b2v)));
+                check(cc_gated_sum(dev, &xv, 1, &yv, opt_view(g1, g1v), opt_view(L.rg1_b, b1v), opt_view(f, fv), opt_view(g2, g2v), opt_view(L.rg2_b, b2v)));
             }
             if (L.side_table.valid()) {
                 CudaTensor g = L.side_gate.matmul_vec(x);
@@ -237,7 +180,11 @@ extern "C" CC_API int cmr_runner_create(cc_device* dev, const cmr_config* conf, 
             const int64_t qh = c.dim + c.rot_dim, hv = (int64_t)c.heads * c.vdim;
             L.norm1 = need(w.norm1, "norm1", {D});
             L.dq_norm = need(w.dq_norm, "mix.dq.norm", {c.q_rank}); L.uq = need(w.uq, "mix.uq", {c.heads * qh, c.q_rank});
-            L.dkv_norm = need(w.dkv_norm, "mix.dkv.norm", {c.kv_rank});
+            if (!w.dkv_norm) throw TensorError(at + "tensor 'mix.dkv.norm' is missing");
+            crabml::LatentAttention& a = L.att;
+            a.heads = c.heads; a.dim = c.dim; a.rot_dim = c.rot_dim; a.vdim = c.vdim; a.kv_rank = c.kv_rank; a.window = c.window; a.scale = c.scale; a.rot_mag = c.rot_mag;
+            a.norm_eps = conf->norm_eps;
+            a.set_weights(dev, at, w.uk, w.uv, w.uk_t, w.uv_f32, w.dkv_norm, w.sink, w.rot_freq);
             L.rg1_b = maybe(w.rg1_b, {D}); L.rg2_b = maybe(w.rg2_b, {D});
             if (c.ff_kind == CMR_FF_NONE && L.rg2_b.valid()) throw TensorError(at + "a gate for a feed-forward the layer does not have");
             L.widths = {c.kv_rank + c.rot_dim, c.q_rank};
@@ -247,16 +194,7 @@ extern "C" CC_API int cmr_runner_create(cc_device* dev, const cmr_config* conf, 
             int64_t on_h = 0;
             for (int32_t v : L.widths) on_h += v;
             L.h_stack = need(w.h_stack, "the stack of mix.dkv, mix.dq, rg1, rg2, mlp.up", {on_h, D});
-            L.uk = need(w.uk, "mix.uk", {(int64_t)c.heads * c.dim, c.kv_rank}); L.uv = need(w.uv, "mix.uv", {hv, c.kv_rank});
-            L.uk_t = need(w.uk_t, "mix.uk (per head transposed)", {(int64_t)c.heads * c.kv_rank, c.dim}); L.uv_f32 = need(w.uv_f32, "mix.uv (F32)", {hv, c.kv_rank});
             L.o = need(w.o, "mix.o", {D, hv});
-            L.sink = maybe(w.sink, {c.heads});
-            if (w.rot_freq) {
-                const int64_t pairs = cc_tensor_capacity(w.rot_freq);
-                if (2 * pairs > c.rot_dim) throw TensorError(at + "more rotated pairs than the rotated part holds");
-                L.rot_freq = CudaTensor::wrap(dev, w.rot_freq, {pairs});
-            }
-            if (L.uk_t.dtype() != CC_F32 || L.uv_f32.dtype() != CC_F32) throw TensorError(at + "the folded forms of mix.uk / mix.uv must be F32: they enter the 32-bit scores and sums");
             if (c.ff_kind == CMR_FF_DENSE) {
                 L.down = need(w.down, "mlp.down", {D, c.ff}); L.act = need(w.act, "mlp.act", {4});
             } else if (c.ff_kind == CMR_FF_ROUTED) {
@@ -272,8 +210,7 @@ extern "C" CC_API int cmr_runner_create(cc_device* dev, const cmr_config* conf, 
                 L.side_gate = need(w.side_gate, "side.gate", {conf->side_dim, D}); L.side_proj = need(w.side_proj, "side.proj", {D, conf->side_dim});
                 L.side_norm = need(w.side_norm, "side.norm", {D});
             }
-            // a ring holds the window's reach behind the first token of a pass, plus the pass
-            L.ring = c.window > 0 ? (int64_t)c.window - 1 + r->conf.chunk : std::max<int64_t>(r->conf.max_seq, r->conf.chunk);
+            L.ring = a.ring_rows(r->conf.chunk, r->conf.max_seq);
         }
         // the order of the runs
         const int n = conf->n_layers;

@@ -7,14 +7,14 @@
 //   pair:   ONE product of the stacked projections (+ biases), cut into its parts ; left: (q, k norms) ; rotation ; keys and values into the
 //           run's rings ; masked softmax (+ sink) ; (sigmoid gate) ; W_o.  right: the recurrence on the run's state ; per-head norm and gate
 //           ; W_o.  Then left_scale * left + right_scale * right.
-//   state space: in-projection cut into z | x B C | dt ; convolution + silu ; scan ; gate, then group norm ; W_o
+//   state space: mixers.hpp
 //   ff:     one product [gate ; up] ; silu(gate + b) * (up + b) ; W_down + b
 #include <cmath>
 #include <string>
 #include <vector>
 
 #include "../../../include/crabml_vuzinex.h"
-#include "seq_runner.hpp"
+#include "mixers.hpp"
 
 using crabml::CudaTensor;
 using crabml::TensorError;
@@ -23,8 +23,9 @@ namespace {
 
 struct Layer {
     cvr_layer_config c{};
-    CudaTensor norm_a, norm_b, norm_c, norm_d, h_stack, h_bias, q_norm, k_norm, sink, rot_freq, left_o, right_norm, right_o, gate_bias_i, gate_bias_f, decay_up, decay_bias, in,
-        conv, conv_bias, dt_bias, a_log, d_skip, s_norm, s_o, gate_up, gate_up_bias, down, down_bias;
+    CudaTensor norm_a, norm_b, norm_c, norm_d, h_stack, h_bias, q_norm, k_norm, sink, rot_freq, left_o, right_norm, right_o, gate_bias_i, gate_bias_f, decay_up, decay_bias,
+        gate_up, gate_up_bias, down, down_bias;
+    crabml::StateSpace ss;
     std::vector<int32_t> widths;         // column blocks of the stacked product, in order
     int i_gate = -1, i_right = 0;        // block of the left gate (-1: none); first block of the right mixer
     int64_t ring = 0;                    // pair: rows of the key / value rings of one run
@@ -36,11 +37,7 @@ struct State : crabml::SeqState {
     std::vector<RunState> runs;
     CudaTensor last;                     // I32 [1]: 1 + the sequence's last token, 0 before the first
 };
-const cc_view* opt(const CudaTensor& t, cc_view& store) {
-    if (!t.valid()) return nullptr;
-    store = t.view();
-    return &store;
-}
+using crabml::opt_view;
 
 struct Runner : csr_runner {
     cvr_config conf{};
@@ -64,8 +61,8 @@ struct Runner : csr_runner {
                     r.S = CudaTensor::alloc({c.r_heads, c.r_dim, c.r_vdim}, CC_F32, dev);
                 }
             } else {
-                r.S = CudaTensor::alloc({c.s_heads, c.s_state, c.s_vdim}, CC_F32, dev);
-                if (c.s_conv > 1) r.tail = CudaTensor::alloc({c.s_conv - 1, (int64_t)c.s_heads * c.s_vdim + 2 * (int64_t)c.s_groups * c.s_state}, CC_F32, dev);
+                r.S = L.ss.make_matrix(dev);
+                r.tail = L.ss.make_tail(dev);
             }
             s->runs.push_back(std::move(r));
         }
@@ -93,15 +90,6 @@ struct Runner : csr_runner {
         cc_view xv = x.view(), yv = y.view(), wv = w.view();
         check(cc_rms_norm_gain_mult(dev, &xv, &yv, &wv, conf.norm_eps, conf.residual_mult));
     }
-    std::vector<CudaTensor> split(const CudaTensor& all, const std::vector<int32_t>& widths) {
-        cc_view av = all.view();
-        std::vector<cc_buf*> outs(widths.size(), nullptr);
-        check(cc_split_cols(dev, &av, (int32_t)widths.size(), widths.data(), outs.data()));
-        std::vector<CudaTensor> part;
-        for (size_t p = 0; p < outs.size(); p++) part.push_back(adopt(outs[p], {all.shape()[0], widths[p]}));
-        return part;
-    }
-
     CudaTensor pair_mixer(const Layer& L, RunState& st, const CudaTensor& h, int64_t pos0) {
         const auto& c = L.c;
         const int64_t n = h.shape()[0];
@@ -111,7 +99,7 @@ struct Runner : csr_runner {
         {
             CudaTensor all = L.h_stack.matmul_vec(h);
             if (L.h_bias.valid()) { cc_view av = all.view(), bv = L.h_bias.view(); check(cc_add_row_bias(dev, &av, &bv)); }
-            part = split(all, L.widths);
+            part = crabml::split_columns(*this, all, L.widths);
         }
         cc_buf* b = nullptr;
         // ---- left: softmax attention over the run's rings
@@ -130,7 +118,7 @@ struct Runner : csr_runner {
         }
         cc_view krv = st.kring.view(), vrv = st.vring.view();
         check(cc_kv_ring_append(dev, &krv, &vrv, &kv, &vv, nullptr, 0.0f, pos0, c.kv_heads, c.dim, c.vdim));
-        check(cc_masked_attention(dev, &qv, &krv, &vrv, pos0, c.heads, c.kv_heads, c.dim, c.vdim, c.window, c.block, c.scale, opt(L.sink, tmp), &b));
+        check(cc_masked_attention(dev, &qv, &krv, &vrv, pos0, c.heads, c.kv_heads, c.dim, c.vdim, c.window, c.block, c.scale, opt_view(L.sink, tmp), &b));
         CudaTensor ol = adopt(b, {n, (int64_t)c.heads * c.vdim});
         b = nullptr;
         if (L.i_gate >= 0) {
@@ -162,28 +150,11 @@ struct Runner : csr_runner {
         return yl;
     }
 
-    CudaTensor state_space_mixer(const Layer& L, RunState& st, const CudaTensor& h) {
-        const auto& c = L.c;
-        const int64_t n = h.shape()[0], inner = (int64_t)c.s_heads * c.s_vdim;
-        std::vector<CudaTensor> part = split(L.in.matmul_vec(h), L.widths);          // z | x B C | dt
-        cc_view xv = part[1].view(), cw = L.conv.view(), cb{}, tl{};
-        cc_buf* b = nullptr;
-        check(cc_short_conv_bias(dev, &xv, &cw, opt(L.conv_bias, cb), opt(st.tail, tl), CC_ACT_SILU, &b));
-        CudaTensor xc = adopt(b, {n, part[1].shape()[1]});
-        b = nullptr;
-        cc_view xcv = xc.view(), dtv = part[2].view(), db = L.dt_bias.view(), al = L.a_log.view(), ds{}, sv = st.S.view();
-        check(cc_state_space_scan(dev, &xcv, &dtv, &db, &al, opt(L.d_skip, ds), &sv, c.s_heads, c.s_groups, c.s_state, c.s_vdim, &b));
-        CudaTensor y = adopt(b, {n, inner});
-        cc_view yv = y.view(), zv = part[0].view(), nw = L.s_norm.view();
-        check(cc_gated_group_rms_norm(dev, &yv, &yv, &zv, &nw, c.s_norm_groups, conf.norm_eps, CC_ACT_SILU));
-        return L.s_o.matmul_vec(y);
-    }
-
     CudaTensor feed_forward(const Layer& L, const CudaTensor& h) {
         CudaTensor gu = L.gate_up.matmul_vec(h);
         cc_view gv = gu.view(), bv{};
         cc_buf* b = nullptr;
-        check(cc_glu_halves(dev, &gv, opt(L.gate_up_bias, bv), CC_ACT_SILU, &b));
+        check(cc_glu_halves(dev, &gv, opt_view(L.gate_up_bias, bv), CC_ACT_SILU, &b));
         CudaTensor z = adopt(b, {h.shape()[0], L.c.ff});
         CudaTensor y = L.down.matmul_vec(z);
         if (L.down_bias.valid()) { cc_view yv = y.view(), dv = L.down_bias.view(); check(cc_add_row_bias(dev, &yv, &dv)); }
@@ -203,7 +174,7 @@ struct Runner : csr_runner {
             const Layer& L = layers[runs[ri]];
             {
                 CudaTensor h = norm(x, L.norm_a);
-                CudaTensor y = L.c.mixer == CVR_MIXER_PAIR ? pair_mixer(L, s.runs[ri], h, pos0) : state_space_mixer(L, s.runs[ri], h);
+                CudaTensor y = L.c.mixer == CVR_MIXER_PAIR ? pair_mixer(L, s.runs[ri], h, pos0) : L.ss.run(*this, s.runs[ri].S, s.runs[ri].tail, h);
                 add_normed(x, y, L.norm_b);
             }
             if (L.c.ff > 0) {
@@ -306,14 +277,9 @@ extern "C" CC_API int cvr_runner_create(cc_device* dev, const cvr_config* conf, 
                 if (c.block > 0 && (reach == 0 || c.block < reach)) reach = c.block;
                 L.ring = reach > 0 ? reach - 1 + r->conf.chunk : std::max<int64_t>(r->conf.max_seq, r->conf.chunk);
             } else if (c.mixer == CVR_MIXER_STATE_SPACE) {
-                if (c.s_heads < 1 || c.s_vdim < 1 || c.s_state < 1 || c.s_groups < 1 || c.s_heads % c.s_groups || c.s_conv < 1) throw TensorError(at + "bad sizes of the state-space mixer");
-                const int64_t inner = (int64_t)c.s_heads * c.s_vdim, bc = 2 * (int64_t)c.s_groups * c.s_state;
-                if (c.s_norm_groups < 1 || inner % c.s_norm_groups) throw TensorError(at + "the norm's groups do not divide the inner width");
-                L.widths = {(int32_t)inner, (int32_t)(inner + bc), c.s_heads};
-                L.in = need(w.in, "mix.in", {2 * inner + bc + c.s_heads, D});
-                L.conv = need(w.conv, "mix.conv", {inner + bc, c.s_conv}); L.conv_bias = maybe(w.conv_bias, {inner + bc});
-                L.dt_bias = need(w.dt_bias, "mix.dt_bias", {c.s_heads}); L.a_log = need(w.a_log, "mix.A_log", {c.s_heads}); L.d_skip = maybe(w.d_skip, {c.s_heads});
-                L.s_norm = need(w.s_norm, "mix.norm", {inner}); L.s_o = need(w.s_o, "mix.o", {D, inner});
+                crabml::StateSpace& m = L.ss;
+                m.heads = c.s_heads; m.vdim = c.s_vdim; m.state = c.s_state; m.groups = c.s_groups; m.conv = c.s_conv; m.norm_groups = c.s_norm_groups; m.norm_eps = conf->norm_eps;
+                m.set_weights(dev, at, D, w.in, w.conv, w.conv_bias, w.dt_bias, w.a_log, w.d_skip, w.s_norm, w.s_o);
             } else throw TensorError(at + "unknown mixer");
             if (c.ff > 0) {
                 L.norm_c = need(w.norm_c, "norm2", {D}); L.norm_d = need(w.norm_d, "norm2b", {D});
@@ -338,7 +304,7 @@ extern "C" CC_API int cvr_runner_create(cc_device* dev, const cvr_config* conf, 
                 r->state_bytes_per_slot += (L.ring * (int64_t)c.kv_heads * (c.dim + c.vdim) + (int64_t)c.r_heads * c.r_dim * (c.r_vdim + (c.right == CVR_RIGHT_MATRIX_MEMORY ? 1 : 0)) +
                                             (c.right == CVR_RIGHT_MATRIX_MEMORY ? c.r_heads : 0)) * 4;
             else
-                r->state_bytes_per_slot += ((int64_t)c.s_heads * c.s_state * c.s_vdim + (int64_t)(c.s_conv - 1) * ((int64_t)c.s_heads * c.s_vdim + 2 * (int64_t)c.s_groups * c.s_state)) * 4;
+                r->state_bytes_per_slot += L.ss.state_floats() * 4;
         }
         if (conf->hash_buckets > 0) r->state_bytes_per_slot += 4;
     });

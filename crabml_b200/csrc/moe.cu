@@ -5,10 +5,15 @@
 // down projection sums the slots IN SLOT ORDER.  A token's result therefore depends only on the token, never on which other
 // tokens share the call (no atomics, no order that depends on the batch).  BF16 expert weights round the operand row to bfloat16
 // (x for gate / up, the hidden row for down) and accumulate in f32, exactly like cc_matmul_vec does for BF16 matrices.
+//
+// A shared expert (every token uses it) is a few more slots: cut into pieces of the experts' hidden width -- its activation works element by
+// element and its down projection adds over the hidden units, so the pieces' results add up to the whole's -- stacked behind the experts and
+// given the weight of the token's shared gate by the router.
 #include <cuda_bf16.h>
 #include <stdlib.h>
 
 #include "../../include/crabml_seqops.h"
+#include "act.cuh"
 #include "capi_checks.cuh"
 
 #define MOE_ENTER(dev, what)                                                                                          \
@@ -37,7 +42,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 // one CTA per token: its warps share the experts' logits (a warp per expert, lanes striding D), then warp 0 does the softmax and the choice
 __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const float* __restrict__ x, const float* __restrict__ wr, const float* __restrict__ corr,
                                                                   int* __restrict__ ids, float* __restrict__ wts, int T, int D, int E, int top, int n_groups, int keep,
-                                                                  int renorm, int score_fn, int group_top, float renorm_eps) {
+                                                                  int renorm, int score_fn, int group_top, float renorm_eps, float scale, const float* __restrict__ wsg, int n_shared) {
     extern __shared__ float rt_sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
@@ -45,12 +50,13 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const float* _
     float* c = s + E;
     float* gs = c + E;
     const float* xr = x + (int64_t)t * D;
-    for (int e = warp; e < E; e += RT_WARPS) {
-        const float* w = wr + (int64_t)e * D;
+    __shared__ float sg;                                   // the shared gate's logit: row E of the same products
+    for (int e = warp; e < E + (wsg ? 1 : 0); e += RT_WARPS) {
+        const float* w = e < E ? wr + (int64_t)e * D : wsg;
         float acc = 0.0f;
         for (int d = lane; d < D; d += 32) acc = fmaf(w[d], xr[d], acc);
         acc = warp_sum(acc);
-        if (lane == 0) s[e] = acc;
+        if (lane == 0) *(e < E ? s + e : &sg) = acc;
     }
     __syncthreads();
     if (warp != 0) return;
@@ -98,24 +104,33 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const float* _
         __syncwarp();
     }
     float wsum = 0.0f;
+    const int slots = top + n_shared;
     for (int r = 0; r < top; r++) {
         float bv = -INFINITY; int bi = 0x7fffffff;
         for (int e = lane; e < E; e += 32) { const float v = c[e]; if (v > bv) { bv = v; bi = e; } }
         warp_argmax(bv, bi);
         if (bi == 0x7fffffff) bi = 0;                       // unreachable with finite scores (keep * group size >= top); never index out of range
         if (lane == 0) {
-            ids[(int64_t)t * top + r] = bi;
-            wts[(int64_t)t * top + r] = s[bi];
+            ids[(int64_t)t * slots + r] = bi;
+            wts[(int64_t)t * slots + r] = s[bi];
             c[bi] = -INFINITY;
         }
         wsum += s[bi];
         __syncwarp();
     }
-    if (renorm && lane == 0) for (int r = 0; r < top; r++) wts[(int64_t)t * top + r] /= wsum + renorm_eps;
+    if (lane == 0) {
+        if (renorm) for (int r = 0; r < top; r++) wts[(int64_t)t * slots + r] /= wsum + renorm_eps;
+        if (scale != 1.0f) for (int r = 0; r < top; r++) wts[(int64_t)t * slots + r] *= scale;
+    }
+    for (int r = lane; r < n_shared; r += 32) {
+        ids[(int64_t)t * slots + top + r] = E + r;
+        wts[(int64_t)t * slots + top + r] = wsg ? act_sigmoid(sg) : 1.0f;
+    }
 }
-extern "C" CC_API int cc_moe_route_ex(cc_device* dev, const cc_view* x, const cc_view* router_w, const cc_view* correction, const cc_route_params* rp, cc_buf** ids_out,
-                                      cc_buf** weights_out) {
+extern "C" CC_API int cc_moe_route_shared(cc_device* dev, const cc_view* x, const cc_view* router_w, const cc_view* correction, const cc_view* shared_gate, int32_t n_shared,
+                                          const cc_route_params* rp, cc_buf** ids_out, cc_buf** weights_out) {
     MOE_ENTER(dev, "moe_route");
+    CC_REQUIRE(dev, n_shared >= 0 && (n_shared > 0 || !shared_gate), "moe_route: %d shared slots", n_shared);
     if (!rp) return cc_fail(dev, CC_ERR_ARG, "moe_route: no parameters");
     int32_t top = rp->top, n_groups = rp->n_groups, keep_groups = rp->keep_groups;
     const int32_t renormalise = rp->renormalise, group_top = rp->group_top < 1 ? 1 : rp->group_top;
@@ -126,13 +141,15 @@ extern "C" CC_API int cc_moe_route_ex(cc_device* dev, const cc_view* x, const cc
     CC_REQUIRE(dev, x->ndim == 2 && router_w->ndim == 2 && router_w->shape[1] == x->shape[1], "moe_route: x must be [T, D] and router_w [E, D]");
     const int64_t T = x->shape[0], D = x->shape[1], E = router_w->shape[0];
     if (correction) { MOE_VIEW(dev, correction, "moe_route correction"); REQUIRE_F32(dev, correction, "moe_route correction"); CC_REQUIRE(dev, view_len(correction) == E, "moe_route: correction must have one number per expert"); }
+    if (shared_gate) { MOE_VIEW(dev, shared_gate, "moe_route shared_gate"); REQUIRE_F32(dev, shared_gate, "moe_route shared_gate"); CC_REQUIRE(dev, view_len(shared_gate) == D, "moe_route: shared_gate must have one number per column of x"); }
+    const float scale = rp->scale == 0.0f ? 1.0f : rp->scale;
     if (n_groups <= 1) { n_groups = 1; keep_groups = 1; }
     CC_REQUIRE(dev, top >= 1 && top <= E && E % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups && (int64_t)keep_groups * (E / n_groups) >= top,
                "moe_route: experts=%lld top=%d groups=%d keep=%d do not fit", (long long)E, top, n_groups, keep_groups);
     cc_buf *ids = nullptr, *wts = nullptr;
-    int rc = cc_new_activation(dev, T * top, CC_I32, false, &ids);
+    int rc = cc_new_activation(dev, T * (top + n_shared), CC_I32, false, &ids);
     if (rc) return rc;
-    rc = cc_new_activation(dev, T * top, CC_F32, false, &wts);
+    rc = cc_new_activation(dev, T * (top + n_shared), CC_F32, false, &wts);
     if (rc) { cc_tensor_release(ids); return rc; }
     *ids_out = ids; *weights_out = wts;
     if (T == 0) return CC_OK;
@@ -142,13 +159,18 @@ extern "C" CC_API int cc_moe_route_ex(cc_device* dev, const cc_view* x, const cc
     moe_route_kernel<<<(unsigned)T, RT_WARPS * 32, smem, dev->stream>>>((const float*)x->buf->plane[0], (const float*)router_w->buf->plane[0],
                                                                                                      correction ? (const float*)correction->buf->plane[0] : nullptr,
                                                                                                      (int*)ids->base, (float*)wts->base, (int)T, (int)D, (int)E, top, n_groups,
-                                                                                                     keep_groups, renormalise, rp->score, group_top, rp->renorm_eps);
+                                                                                                     keep_groups, renormalise, rp->score, group_top, rp->renorm_eps, scale,
+                                                                                                     shared_gate ? (const float*)shared_gate->buf->plane[0] : nullptr, n_shared);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
+extern "C" CC_API int cc_moe_route_ex(cc_device* dev, const cc_view* x, const cc_view* router_w, const cc_view* correction, const cc_route_params* rp, cc_buf** ids_out,
+                                      cc_buf** weights_out) {
+    return cc_moe_route_shared(dev, x, router_w, correction, nullptr, 0, rp, ids_out, weights_out);
+}
 extern "C" CC_API int cc_moe_route(cc_device* dev, const cc_view* x, const cc_view* router_w, const cc_view* correction, int32_t top, int32_t n_groups,
                                    int32_t keep_groups, int32_t renormalise, cc_buf** ids_out, cc_buf** weights_out) {
-    const cc_route_params rp = {CC_ROUTE_SOFTMAX, top, n_groups, keep_groups, 1, renormalise, 0.0f};
+    const cc_route_params rp = {CC_ROUTE_SOFTMAX, top, n_groups, keep_groups, 1, renormalise, 0.0f, 1.0f};
     return cc_moe_route_ex(dev, x, router_w, correction, &rp, ids_out, weights_out);
 }
 
@@ -161,38 +183,60 @@ template <class WT> __device__ __forceinline__ float moe_round(float v);
 template <> __device__ __forceinline__ float moe_round<float>(float v) { return v; }
 template <> __device__ __forceinline__ float moe_round<uint16_t>(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 
-__device__ __forceinline__ float moe_act(float z, int act, float alpha) {
-    return act == CC_ACT_SILU ? z / (1.0f + expf(-z)) : act == CC_ACT_GELU_TANH ? 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)))
-         : act == CC_ACT_SWISH ? z / (1.0f + expf(-(alpha * z))) : z;
-}
 // the gated unit: act(min(g, limit)) * (clamp(u, -limit, limit) + up_shift); limit <= 0 clamps nothing
 __device__ __forceinline__ float moe_glu(float g, float u, const cc_glu_params P) {
     if (P.limit > 0.0f) { g = fminf(g, P.limit); u = fminf(fmaxf(u, -P.limit), P.limit); }
-    return moe_act(g, P.act, P.alpha) * (u + P.up_shift);
+    return act_apply(g, P.act, P.alpha) * (u + P.up_shift);
 }
 
-// grid (T * top, ceil(ff / 8)), 256 threads: the CTA stages x[t] (rounded for BF16 weights); a warp owns one hidden row of the slot's expert
-template <class WT>
+// one lane's share of a row's dot product with a vector in shared memory.  VEC: 16-byte pieces (4 floats or 8 bfloat16) of the row, lane-strided;
+// else element by element
+template <class WT, bool VEC> __device__ __forceinline__ float moe_dot(const WT* __restrict__ w, const float* xs, int n, int lane) {
+    float acc = 0.0f;
+    if (!VEC) {
+        for (int d = lane; d < n; d += 32) acc = fmaf(moe_w(w, d), xs[d], acc);
+    } else if (sizeof(WT) == 4) {
+#pragma unroll 4
+        for (int d = lane * 4; d < n; d += 128) {
+            const float4 v = *(const float4*)(w + d), x = *(const float4*)(xs + d);
+            acc = fmaf(v.x, x.x, acc); acc = fmaf(v.y, x.y, acc); acc = fmaf(v.z, x.z, acc); acc = fmaf(v.w, x.w, acc);
+        }
+    } else {
+#pragma unroll 4
+        for (int d = lane * 8; d < n; d += 256) {
+            const uint4 v = *(const uint4*)(w + d);
+            const float4 x = *(const float4*)(xs + d), y = *(const float4*)(xs + d + 4);
+            acc = fmaf(__uint_as_float(v.x << 16), x.x, acc); acc = fmaf(__uint_as_float(v.x & 0xffff0000u), x.y, acc);
+            acc = fmaf(__uint_as_float(v.y << 16), x.z, acc); acc = fmaf(__uint_as_float(v.y & 0xffff0000u), x.w, acc);
+            acc = fmaf(__uint_as_float(v.z << 16), y.x, acc); acc = fmaf(__uint_as_float(v.z & 0xffff0000u), y.y, acc);
+            acc = fmaf(__uint_as_float(v.w << 16), y.z, acc); acc = fmaf(__uint_as_float(v.w & 0xffff0000u), y.w, acc);
+        }
+    }
+    return acc;
+}
+// grid (T * top, ceil(ff / 8)), 256 threads: the CTA stages x[t] (rounded for BF16 weights); a warp owns one hidden row of the slot's expert.
+// wg NULL: a plain unit, act(W_up x); ids NULL: every slot is expert 0 (a dense feed-forward)
+template <class WT, bool VEC>
 __global__ void __launch_bounds__(256) moe_gate_up_kernel(const float* __restrict__ x, const int* __restrict__ ids, const WT* __restrict__ wg, const WT* __restrict__ wu,
                                                           float* __restrict__ hid, int D, int ff, int top, cc_glu_params act, int E) {
-    extern __shared__ float mg_sm[];
+    extern __shared__ __align__(16) float mg_sm[];
     const int ts = blockIdx.x, t = ts / top;
-    const int e = moe_clamp(ids[ts], E);
+    const int e = ids ? moe_clamp(ids[ts], E) : 0;
     for (int d = threadIdx.x; d < D; d += 256) mg_sm[d] = moe_round<WT>(x[(int64_t)t * D + d]);
     __syncthreads();
     const int r = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (r >= ff) return;
     const int64_t base = ((int64_t)e * ff + r) * D;
-    float g = 0.0f, u = 0.0f;
-    for (int d = lane; d < D; d += 32) { const float xv = mg_sm[d]; g = fmaf(moe_w(wg, base + d), xv, g); u = fmaf(moe_w(wu, base + d), xv, u); }
-    g = warp_sum(g); u = warp_sum(u);
-    if (lane == 0) hid[(int64_t)ts * ff + r] = moe_glu(g, u, act);
+    float g = wg ? moe_dot<WT, VEC>(wg + base, mg_sm, D, lane) : 0.0f, u = moe_dot<WT, VEC>(wu + base, mg_sm, D, lane);
+    if (wg) g = warp_sum(g);
+    u = warp_sum(u);
+    if (lane == 0) hid[(int64_t)ts * ff + r] = wg ? moe_glu(g, u, act) : act_apply(u, act.act, act.alpha);
 }
 // grid (T, ceil(D / 8)), 256 threads: the CTA stages the token's top hidden rows; a warp owns one output coordinate and adds the slots in order
-template <class WT>
+template <class WT, bool VEC>
 __global__ void __launch_bounds__(256) moe_down_kernel(const float* __restrict__ hid, const int* __restrict__ ids, const float* __restrict__ wts, const WT* __restrict__ wd,
                                                        float* __restrict__ out, int D, int ff, int top, int E) {
-    extern __shared__ float md_sm[];
+    extern __shared__ __align__(16) float md_sm[];
     const int t = blockIdx.x;
     for (int i = threadIdx.x; i < top * ff; i += 256) md_sm[i] = moe_round<WT>(hid[(int64_t)t * top * ff + i]);
     __syncthreads();
@@ -200,28 +244,33 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const float* __restrict__
     if (d >= D) return;
     float acc = 0.0f;
     for (int s = 0; s < top; s++) {
-        const int e = moe_clamp(ids[(int64_t)t * top + s], E);
-        const int64_t base = ((int64_t)e * D + d) * ff;
-        float p = 0.0f;
-        for (int f = lane; f < ff; f += 32) p = fmaf(moe_w(wd, base + f), md_sm[s * ff + f], p);
-        p = warp_sum(p);
-        acc = fmaf(wts[(int64_t)t * top + s], p, acc);
+        const int e = ids ? moe_clamp(ids[(int64_t)t * top + s], E) : 0;
+        const float p = warp_sum(moe_dot<WT, VEC>(wd + ((int64_t)e * D + d) * ff, md_sm + s * ff, ff, lane));
+        acc = wts ? fmaf(wts[(int64_t)t * top + s], p, acc) : acc + p;
     }
     if (lane == 0) out[(int64_t)t * D + d] = acc;
 }
 
+template <class WT, bool VEC>
+static int moe_launch_vec(cc_device* dev, const float* x, const int* ids, const float* wts, const WT* wg, const WT* wu, const WT* wd, float* hid, float* out, int64_t T,
+                          int D, int ff, int top, cc_glu_params act, int E) {
+    const size_t s1 = (size_t)D * 4, s2 = (size_t)top * ff * 4;
+    if (s1 > 200 * 1024 || s2 > 200 * 1024) return cc_fail(dev, CC_ERR_UNSUPPORTED, "moe_experts: row does not fit shared memory");
+    if (s1 > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_gate_up_kernel<WT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1));
+    if (s2 > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_down_kernel<WT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2));
+    moe_gate_up_kernel<WT, VEC><<<dim3((unsigned)(T * top), (unsigned)((ff + 7) / 8)), 256, s1, dev->stream>>>(x, ids, wg, wu, hid, D, ff, top, act, E);
+    CC_LAUNCH_CHECK(dev);
+    moe_down_kernel<WT, VEC><<<dim3((unsigned)T, (unsigned)((D + 7) / 8)), 256, s2, dev->stream>>>(hid, ids, wts, wd, out, D, ff, top, E);
+    CC_LAUNCH_CHECK(dev);
+    return CC_OK;
+}
 template <class WT>
 static int moe_launch(cc_device* dev, const float* x, const int* ids, const float* wts, const void* wg, const void* wu, const void* wd, float* hid, float* out, int64_t T,
                       int D, int ff, int top, cc_glu_params act, int E) {
-    const size_t s1 = (size_t)D * 4, s2 = (size_t)top * ff * 4;
-    if (s1 > 200 * 1024 || s2 > 200 * 1024) return cc_fail(dev, CC_ERR_UNSUPPORTED, "moe_experts: row does not fit shared memory");
-    if (s1 > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_gate_up_kernel<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1));
-    if (s2 > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_down_kernel<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2));
-    moe_gate_up_kernel<WT><<<dim3((unsigned)(T * top), (unsigned)((ff + 7) / 8)), 256, s1, dev->stream>>>(x, ids, (const WT*)wg, (const WT*)wu, hid, D, ff, top, act, E);
-    CC_LAUNCH_CHECK(dev);
-    moe_down_kernel<WT><<<dim3((unsigned)T, (unsigned)((D + 7) / 8)), 256, s2, dev->stream>>>(hid, ids, wts, (const WT*)wd, out, D, ff, top, E);
-    CC_LAUNCH_CHECK(dev);
-    return CC_OK;
+    constexpr int per = 16 / (int)sizeof(WT);
+    const bool vec = D % per == 0 && ff % per == 0 && (((uintptr_t)wg | (uintptr_t)wu | (uintptr_t)wd) & 15) == 0;
+    return vec ? moe_launch_vec<WT, true>(dev, x, ids, wts, (const WT*)wg, (const WT*)wu, (const WT*)wd, hid, out, T, D, ff, top, act, E)
+               : moe_launch_vec<WT, false>(dev, x, ids, wts, (const WT*)wg, (const WT*)wu, (const WT*)wd, hid, out, T, D, ff, top, act, E);
 }
 
 // ---- grouped path (BF16 weights, many rows): the (token, slot) rows are sorted by expert and every expert's rows run through the
@@ -267,7 +316,17 @@ __global__ void moe_gather_bf16_kernel(const float* __restrict__ x, const int* _
 __global__ void moe_glu_bf16_kernel(const float* __restrict__ g, const float* __restrict__ u, __nv_bfloat16* __restrict__ h, int64_t n, cc_glu_params act) {
     const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 2;
     if (i >= n) return;
-    *(__nv_bfloat162*)(h + i) = __floats2bfloat162_rn(moe_glu(g[i], u[i], act), moe_glu(g[i + 1], u[i + 1], act));
+    const float2 uv = *(const float2*)(u + i);
+    if (g) {
+        const float2 gv = *(const float2*)(g + i);
+        *(__nv_bfloat162*)(h + i) = __floats2bfloat162_rn(moe_glu(gv.x, uv.x, act), moe_glu(gv.y, uv.y, act));
+    } else {                                                  // a plain unit: act(u)
+        *(__nv_bfloat162*)(h + i) = __floats2bfloat162_rn(act_apply(uv.x, act.act, act.alpha), act_apply(uv.y, act.act, act.alpha));
+    }
+}
+__global__ void moe_activate_kernel(float* __restrict__ x, int64_t n, int act) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = act_apply(x[i], act);
 }
 // out[t][d] = sum over the slots, in slot order, of weights[t][s] * y[pos[t * top + s]][d]
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ wts, float* __restrict__ out, int64_t T, int top, int D) {
@@ -286,19 +345,19 @@ static int moe_grouped(cc_device* dev, const float* x, const int* ids, const flo
     const int max_tiles = (int)((n + block_n - 1) / block_n) + E;
     // one pool block: pos[n] | table[4 + 4 * max_tiles] | xs bf16 [n][D] | g f32 [n][ff] | u f32 [n][ff] | h bf16 [n][ff] | y f32 [n][D]
     auto al = [](size_t v) { return (v + 255) & ~(size_t)255; };
-    const size_t o_pos = 0, o_tab = al((size_t)n * 4), o_xs = o_tab + al((size_t)(4 + 4 * max_tiles) * 4), o_g = o_xs + al((size_t)n * D * 2), o_u = o_g + al((size_t)n * ff * 4),
+    const size_t o_pos = 0, o_tab = al((size_t)n * 4), o_xs = o_tab + al((size_t)(4 + 4 * max_tiles) * 4), o_g = o_xs + al((size_t)n * D * 2), o_u = o_g + (wg ? al((size_t)n * ff * 4) : 0),
                  o_h = o_u + al((size_t)n * ff * 4), o_y = o_h + al((size_t)n * ff * 2), total = o_y + al((size_t)n * D * 4);
     uint8_t* base = nullptr; size_t cls = 0;
     int rc = cc_pool_alloc(dev, total, (void**)&base, &cls);
     if (rc) return rc;
     int* pos = (int*)(base + o_pos); int* table = (int*)(base + o_tab);
-    __nv_bfloat16* xs = (__nv_bfloat16*)(base + o_xs); float* g = (float*)(base + o_g); float* u = (float*)(base + o_u);
+    __nv_bfloat16* xs = (__nv_bfloat16*)(base + o_xs); float* g = wg ? (float*)(base + o_g) : nullptr; float* u = (float*)(base + o_u);
     __nv_bfloat16* h = (__nv_bfloat16*)(base + o_h); float* y = (float*)(base + o_y);
     moe_sort_kernel<<<1, 1024, (size_t)2 * E * 4, dev->stream>>>(ids, (int)n, E, block_n, pos, table);
     dev->launches++;
     moe_gather_bf16_kernel<<<(unsigned)((n + 7) / 8), 256, 0, dev->stream>>>(x, pos, xs, (int)n, top, D);
     dev->launches++;
-    rc = cc_launch_grouped_bf16(dev, wg, E, ff, D, xs, n, table, max_tiles, block_n, g);
+    if (wg) rc = cc_launch_grouped_bf16(dev, wg, E, ff, D, xs, n, table, max_tiles, block_n, g);
     if (!rc) rc = cc_launch_grouped_bf16(dev, wu, E, ff, D, xs, n, table, max_tiles, block_n, u);
     if (!rc) {
         moe_glu_bf16_kernel<<<(unsigned)((n * ff / 2 + 255) / 256), 256, 0, dev->stream>>>(g, u, h, n * ff, act);
@@ -313,21 +372,25 @@ static int moe_grouped(cc_device* dev, const float* x, const int* ids, const flo
     return rc;
 }
 
-extern "C" CC_API int cc_moe_experts_glu(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_gate, const cc_view* w_up,
-                                         const cc_view* w_down, int32_t n_experts, int32_t ff, const cc_glu_params* glu, cc_buf** out) {
+// w_gate NULL: plain units, act(W_up x); ids NULL (with weights NULL): no router, every token runs the one expert with weight 1
+static int moe_experts_impl(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_gate, const cc_view* w_up, const cc_view* w_down,
+                            int32_t n_experts, int32_t ff, const cc_glu_params act, cc_buf** out) {
     MOE_ENTER(dev, "moe_experts");
-    if (!glu) return cc_fail(dev, CC_ERR_ARG, "moe_experts: no gated-unit parameters");
-    const cc_glu_params act = *glu;
     if (!out) return cc_fail(dev, CC_ERR_ARG, "moe_experts: out is NULL");
-    MOE_VIEW(dev, x, "moe_experts x"); MOE_VIEW(dev, ids, "moe_experts ids"); MOE_VIEW(dev, weights, "moe_experts weights");
-    MOE_VIEW(dev, w_gate, "moe_experts w_gate"); MOE_VIEW(dev, w_up, "moe_experts w_up"); MOE_VIEW(dev, w_down, "moe_experts w_down");
-    REQUIRE_F32(dev, x, "moe_experts x"); REQUIRE_F32(dev, weights, "moe_experts weights");
-    CC_REQUIRE(dev, ids->buf->dtype == CC_I32, "moe_experts: ids must be I32");
-    CC_REQUIRE(dev, x->ndim == 2 && ids->ndim == 2 && ids->shape[0] == x->shape[0] && view_len(weights) == view_len(ids), "moe_experts: x must be [T, D], ids and weights [T, top]");
-    const int64_t T = x->shape[0], D = x->shape[1], top = ids->shape[1];
-    const int wt = w_gate->buf->dtype;
-    CC_REQUIRE(dev, (wt == CC_F32 || wt == CC_BF16) && w_up->buf->dtype == wt && w_down->buf->dtype == wt, "moe_experts: expert weights must all be F32 or all BF16");
-    CC_REQUIRE(dev, n_experts > 0 && ff > 0 && view_len(w_gate) == (int64_t)n_experts * ff * D && view_len(w_up) == (int64_t)n_experts * ff * D &&
+    MOE_VIEW(dev, x, "moe_experts x"); MOE_VIEW(dev, w_up, "moe_experts w_up"); MOE_VIEW(dev, w_down, "moe_experts w_down");
+    if (w_gate) MOE_VIEW(dev, w_gate, "moe_experts w_gate");
+    REQUIRE_F32(dev, x, "moe_experts x");
+    CC_REQUIRE(dev, x->ndim == 2, "moe_experts: x must be [T, D]");
+    if (ids) {
+        MOE_VIEW(dev, ids, "moe_experts ids"); MOE_VIEW(dev, weights, "moe_experts weights");
+        REQUIRE_F32(dev, weights, "moe_experts weights");
+        CC_REQUIRE(dev, ids->buf->dtype == CC_I32, "moe_experts: ids must be I32");
+        CC_REQUIRE(dev, ids->ndim == 2 && ids->shape[0] == x->shape[0] && view_len(weights) == view_len(ids), "moe_experts: x must be [T, D], ids and weights [T, top]");
+    }
+    const int64_t T = x->shape[0], D = x->shape[1], top = ids ? ids->shape[1] : 1;
+    const int wt = w_up->buf->dtype;
+    CC_REQUIRE(dev, (wt == CC_F32 || wt == CC_BF16) && (!w_gate || w_gate->buf->dtype == wt) && w_down->buf->dtype == wt, "moe_experts: expert weights must all be F32 or all BF16");
+    CC_REQUIRE(dev, n_experts > 0 && ff > 0 && (!w_gate || view_len(w_gate) == (int64_t)n_experts * ff * D) && view_len(w_up) == (int64_t)n_experts * ff * D &&
                         view_len(w_down) == (int64_t)n_experts * D * ff,
                "moe_experts: weight stacks do not fit experts=%d ff=%d D=%lld", n_experts, ff, (long long)D);
     cc_buf* o = nullptr;
@@ -335,24 +398,72 @@ extern "C" CC_API int cc_moe_experts_glu(cc_device* dev, const cc_view* x, const
     if (rc) return rc;
     *out = o;
     if (T == 0) return CC_OK;
+    const float* xp = (const float*)x->buf->plane[0];
+    const int* ip = ids ? (const int*)ids->buf->plane[0] : nullptr;
+    const float* wp = ids ? (const float*)weights->buf->plane[0] : nullptr;
+    const void *gp = w_gate ? w_gate->buf->plane[0] : nullptr, *up = w_up->buf->plane[0], *dp = w_down->buf->plane[0];
     static const int grouped_min_rows = getenv("CRABML_MOE_GROUPED_MIN") ? atoi(getenv("CRABML_MOE_GROUPED_MIN")) : 128;
-    if (wt == CC_BF16 && T * top >= grouped_min_rows && n_experts <= 4096 && D % 2 == 0 && ff % 2 == 0 && cc_grouped_bf16_supported(ff, D) && cc_grouped_bf16_supported(D, ff) &&
-        ((uintptr_t)w_gate->buf->plane[0] & 15) == 0 && ((uintptr_t)w_up->buf->plane[0] & 15) == 0 && ((uintptr_t)w_down->buf->plane[0] & 15) == 0)
-        return moe_grouped(dev, (const float*)x->buf->plane[0], (const int*)ids->buf->plane[0], (const float*)weights->buf->plane[0], w_gate->buf, w_up->buf, w_down->buf,
-                           (float*)o->base, T, (int)D, ff, (int)top, n_experts, act);
+    if (ids && wt == CC_BF16 && T * top >= grouped_min_rows && n_experts <= 4096 && D % 2 == 0 && ff % 2 == 0 && cc_grouped_bf16_supported(ff, D) && cc_grouped_bf16_supported(D, ff) &&
+        (((uintptr_t)gp | (uintptr_t)up | (uintptr_t)dp) & 15) == 0)
+        return moe_grouped(dev, xp, ip, wp, w_gate ? w_gate->buf : nullptr, w_up->buf, w_down->buf, (float*)o->base, T, (int)D, ff, (int)top, n_experts, act);
     void* hid = nullptr; size_t cls = 0;
     rc = cc_pool_alloc(dev, (size_t)T * top * ff * 4, &hid, &cls);
     if (rc) return rc;
-    const float* xp = (const float*)x->buf->plane[0];
-    const int* ip = (const int*)ids->buf->plane[0];
-    const float* wp = (const float*)weights->buf->plane[0];
-    if (wt == CC_F32) rc = moe_launch<float>(dev, xp, ip, wp, w_gate->buf->plane[0], w_up->buf->plane[0], w_down->buf->plane[0], (float*)hid, (float*)o->base, T, (int)D, ff, (int)top, act, n_experts);
-    else rc = moe_launch<uint16_t>(dev, xp, ip, wp, w_gate->buf->plane[0], w_up->buf->plane[0], w_down->buf->plane[0], (float*)hid, (float*)o->base, T, (int)D, ff, (int)top, act, n_experts);
+    if (wt == CC_F32) rc = moe_launch<float>(dev, xp, ip, wp, gp, up, dp, (float*)hid, (float*)o->base, T, (int)D, ff, (int)top, act, n_experts);
+    else rc = moe_launch<uint16_t>(dev, xp, ip, wp, gp, up, dp, (float*)hid, (float*)o->base, T, (int)D, ff, (int)top, act, n_experts);
     cc_pool_free(dev, hid, cls);
     return rc;
+}
+extern "C" CC_API int cc_moe_experts_glu(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_gate, const cc_view* w_up,
+                                         const cc_view* w_down, int32_t n_experts, int32_t ff, const cc_glu_params* glu, cc_buf** out) {
+    if (dev && (!glu || !w_gate || !ids || !weights)) return cc_fail(dev, CC_ERR_ARG, "moe_experts: an operand is NULL");
+    return moe_experts_impl(dev, x, ids, weights, w_gate, w_up, w_down, n_experts, ff, dev ? *glu : cc_glu_params{}, out);
 }
 extern "C" CC_API int cc_moe_experts(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_gate, const cc_view* w_up,
                                      const cc_view* w_down, int32_t n_experts, int32_t ff, int32_t act, cc_buf** out) {
     const cc_glu_params glu = {act, 1.0f, 0.0f, 0.0f};
     return cc_moe_experts_glu(dev, x, ids, weights, w_gate, w_up, w_down, n_experts, ff, &glu, out);
+}
+extern "C" CC_API int cc_moe_experts_act(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_up, const cc_view* w_down, int32_t n_experts,
+                                         int32_t ff, int32_t act, cc_buf** out) {
+    if (dev && (!ids || !weights)) return cc_fail(dev, CC_ERR_ARG, "moe_experts: an operand is NULL");
+    return moe_experts_impl(dev, x, ids, weights, nullptr, w_up, w_down, n_experts, ff, cc_glu_params{act, 1.0f, 0.0f, 0.0f}, out);
+}
+
+// ---- a dense feed-forward of plain units ----------------------------------------------------------------------------------------------------
+bool cc_prefill_bf16_supported(int64_t m, int64_t k, int64_t b);                                                                              // prefill_gemm.cu
+int cc_launch_prefill_bf16_act(cc_device* dev, const cc_buf* w, const float* x_f32, int act, float* out, int64_t m, int64_t k, int64_t b);
+bool cc_dense_supported(int wtype, int64_t b);                                                                                                // dense.cu
+int cc_launch_dense(cc_device* dev, const cc_buf* w, const float* x, float* out, int64_t m, int64_t k, int64_t b);
+extern "C" CC_API int cc_feed_forward_act(cc_device* dev, const cc_view* x, const cc_view* w_up, const cc_view* w_down, int32_t act, cc_buf** out) {
+    MOE_ENTER(dev, "feed_forward_act");
+    if (!out) return cc_fail(dev, CC_ERR_ARG, "feed_forward_act: out is NULL");
+    MOE_VIEW(dev, x, "feed_forward_act x"); MOE_VIEW(dev, w_up, "feed_forward_act w_up"); MOE_VIEW(dev, w_down, "feed_forward_act w_down");
+    REQUIRE_F32(dev, x, "feed_forward_act x");
+    CC_REQUIRE(dev, x->ndim == 2 && w_up->ndim == 2 && w_down->ndim == 2 && w_up->shape[1] == x->shape[1] && w_down->shape[0] == x->shape[1] && w_down->shape[1] == w_up->shape[0],
+               "feed_forward_act: x must be [T, D], w_up [ff, D] and w_down [D, ff]");
+    const int64_t T = x->shape[0], D = x->shape[1], ff = w_up->shape[0];
+    const int wt = w_up->buf->dtype;
+    CC_REQUIRE(dev, (wt == CC_F32 || wt == CC_BF16) && w_down->buf->dtype == wt, "feed_forward_act: the weights must both be F32 or both BF16");
+    if (!cc_dense_supported(wt, T)) return moe_experts_impl(dev, x, nullptr, nullptr, nullptr, w_up, w_down, 1, (int32_t)ff, cc_glu_params{act, 1.0f, 0.0f, 0.0f}, out);
+    cc_buf* o = nullptr;
+    int rc = cc_new_activation(dev, T * D, CC_F32, false, &o);
+    if (rc) return rc;
+    *out = o;
+    void* hid = nullptr; size_t cls = 0;
+    rc = cc_pool_alloc(dev, (size_t)T * ff * 4, &hid, &cls);
+    if (rc) return rc;
+    rc = cc_launch_dense(dev, w_up->buf, (const float*)x->buf->plane[0], (float*)hid, ff, D, T);
+    if (!rc) {
+        if (wt == CC_BF16 && cc_prefill_bf16_supported(D, ff, T) && ((uintptr_t)w_down->buf->plane[0] & 15) == 0) {
+            rc = cc_launch_prefill_bf16_act(dev, w_down->buf, (const float*)hid, act, (float*)o->base, D, ff, T);          // the activation rides in the operand's conversion
+        } else {
+            const int64_t n = T * ff;
+            moe_activate_kernel<<<(unsigned)((n + 255) / 256), 256, 0, dev->stream>>>((float*)hid, n, act);
+            dev->launches++;
+            rc = cc_launch_dense(dev, w_down->buf, (const float*)hid, (float*)o->base, D, ff, T);
+        }
+    }
+    cc_pool_free(dev, hid, cls);
+    return rc;
 }

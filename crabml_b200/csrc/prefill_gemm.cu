@@ -21,6 +21,7 @@
 
 #include <cuda_bf16.h>
 
+#include "act.cuh"
 #include "common.cuh"
 #include "dequant.cuh"
 
@@ -362,21 +363,24 @@ int cc_launch_prefill_matmul(cc_device* dev, const cc_buf* w, const void* act_q8
 
 // ---- plain bfloat16 weights (dense.cu): the weight matrix [m][k] is its own tile source, the f32 activation rows are rounded to
 // bfloat16 once, and the same pipeline runs with the bf16 operand format ---------------------------------------------------------------
-__global__ void act_f32_to_bf16_kernel(const float* __restrict__ x, int64_t nelems, __nv_bfloat16* __restrict__ out) {
+// act: an activation applied on the way (CC_ACT_NONE: none), before the rounding
+__global__ void act_f32_to_bf16_kernel(const float* __restrict__ x, int64_t nelems, __nv_bfloat16* __restrict__ out, int act) {
     const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 2;
     if (i >= nelems) return;
-    *(__nv_bfloat162*)(out + i) = __floats2bfloat162_rn(x[i], x[i + 1]);
+    float a = x[i], b = x[i + 1];
+    if (act != CC_ACT_NONE) { a = act_apply(a, act); b = act_apply(b, act); }
+    *(__nv_bfloat162*)(out + i) = __floats2bfloat162_rn(a, b);
 }
 bool cc_prefill_bf16_supported(int64_t m, int64_t k, int64_t b) {
     static const bool off = getenv("CRABML_PREFILL_OFF") != nullptr;
     return !off && b >= 32 && m >= 1 && k >= PG_BLOCK_K && k % PG_BLOCK_K == 0;
 }
-int cc_launch_prefill_bf16(cc_device* dev, const cc_buf* w, const float* x_f32, float* out, int64_t m, int64_t k, int64_t b) {
+int cc_launch_prefill_bf16_act(cc_device* dev, const cc_buf* w, const float* x_f32, int act, float* out, int64_t m, int64_t k, int64_t b) {
     PgScratch* s = pg_scratch(dev);
     int rc = pg_ensure(dev, &s->x, &s->x_bytes, (size_t)b * k * 2);
     if (rc) return rc;
     const int64_t na = b * k;
-    act_f32_to_bf16_kernel<<<(unsigned)((na / 2 + 255) / 256), 256, 0, dev->stream>>>(x_f32, na, (__nv_bfloat16*)s->x);
+    act_f32_to_bf16_kernel<<<(unsigned)((na / 2 + 255) / 256), 256, 0, dev->stream>>>(x_f32, na, (__nv_bfloat16*)s->x, act);
     CC_LAUNCH_CHECK(dev);
     const int block_n = b >= 192 ? 256 : b >= 96 ? 128 : 64;
     CUtensorMap tw, tx;
@@ -388,6 +392,10 @@ int cc_launch_prefill_bf16(cc_device* dev, const cc_buf* w, const float* x_f32, 
     if (block_n == 256) return mt2 ? pg_launch<256, 2, 1>(dev, tw, tx, out, m, b, k) : pg_launch<256, 1, 1>(dev, tw, tx, out, m, b, k);
     if (block_n == 128) return mt2 ? pg_launch<128, 2, 1>(dev, tw, tx, out, m, b, k) : pg_launch<128, 1, 1>(dev, tw, tx, out, m, b, k);
     return mt2 ? pg_launch<64, 2, 1>(dev, tw, tx, out, m, b, k) : pg_launch<64, 1, 1>(dev, tw, tx, out, m, b, k);
+}
+
+int cc_launch_prefill_bf16(cc_device* dev, const cc_buf* w, const float* x_f32, float* out, int64_t m, int64_t k, int64_t b) {
+    return cc_launch_prefill_bf16_act(dev, w, x_f32, CC_ACT_NONE, out, m, k, b);
 }
 
 // ---- grouped products of the routed feed-forward (moe.cu): X rows sorted by group, W = group-major stack [groups * m][k] ------------------

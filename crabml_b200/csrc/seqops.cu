@@ -9,6 +9,7 @@
 #include <cuda_bf16.h>
 
 #include "../../include/crabml_seqops.h"
+#include "act.cuh"
 #include "capi_checks.cuh"
 
 #define SEQ_ENTER(dev, what)                                                                                          \
@@ -27,15 +28,20 @@
         SEQ_VIEW(dev, v, what);              \
         REQUIRE_F32(dev, v, what);           \
     } while (0)
+// rows of a wider matrix (a column block, or the whole): unit column stride, any row stride that holds a row
+#define SEQ_ROWS(dev, v, what)                                                                                        \
+    do {                                                                                                              \
+        if (!view_ok(v)) return cc_fail((dev), CC_ERR_ARG, "%s: bad tensor view", what);                              \
+        if (!view_in_bounds(v)) return cc_fail((dev), CC_ERR_TENSOR, "%s: view addresses element %lld of a buffer of %lld", what, \
+                                               (long long)view_max_offset(v), (long long)(v)->buf->nelems);           \
+        REQUIRE_F32(dev, v, what);                                                                                    \
+        CC_REQUIRE(dev, (v)->ndim == 2 && (v)->strides[1] == 1 && (v)->strides[0] >= (v)->shape[1], "%s: not rows of a matrix", what); \
+    } while (0)
 static inline float* fptr(const cc_view* v) { return (float*)v->buf->plane[0]; }
 
-__device__ __forceinline__ float seq_silu(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float seq_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float seq_sigmoid(float z) { return act_sigmoid(z); }
 __device__ __forceinline__ float seq_softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float seq_gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
-__device__ __forceinline__ float seq_act(float z, int act) {
-    return act == CC_ACT_SILU ? seq_silu(z) : act == CC_ACT_GELU_TANH ? seq_gelu_tanh(z) : act == CC_ACT_SIGMOID ? seq_sigmoid(z) : z;
-}
+__device__ __forceinline__ float seq_act(float z, int act) { return act_apply(z, act); }
 
 extern "C" CC_API int cc_tensor_zero(cc_device* dev, const cc_view* x) {
     SEQ_ENTER(dev, "tensor_zero");
@@ -63,6 +69,28 @@ __global__ void rms_norm_gain_kernel(float* __restrict__ dst, const float* __res
         dr[c] = accumulate ? dr[c] + v : v;
     }
 }
+// a wide row: one CTA per row, so that a call of few rows does not walk it with a single warp.  Thread-strided sums, the butterfly, then the
+// warps' sums in warp order: the order depends on the row's length alone
+#define RNG_THREADS 256
+__global__ void __launch_bounds__(RNG_THREADS) rms_norm_gain_wide_kernel(float* __restrict__ dst, const float* __restrict__ y, const float* __restrict__ gain, int gain_n, int cols,
+                                                                         float eps, int accumulate, float mult) {
+    __shared__ float red[RNG_THREADS / 32];
+    const float* yr = y + (int64_t)blockIdx.x * cols;
+    float* dr = dst + (int64_t)blockIdx.x * cols;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < cols; c += RNG_THREADS) ss = fmaf(yr[c], yr[c], ss);
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float tot = 0.0f;
+#pragma unroll
+    for (int w = 0; w < RNG_THREADS / 32; w++) tot += red[w];
+    const float inv = 1.0f / sqrtf(tot / (float)cols + eps);
+    for (int c = threadIdx.x; c < cols; c += RNG_THREADS) {
+        const float v = yr[c] * inv * gain[gain_n == 1 ? 0 : c] * mult;
+        dr[c] = accumulate ? dr[c] + v : v;
+    }
+}
 static int rms_norm_gain_impl(cc_device* dev, const cc_view* dst, const cc_view* y, const cc_view* gain, float eps, int32_t accumulate, float mult) {
     SEQ_ENTER(dev, "rms_norm_gain");
     SEQ_F32(dev, dst, "rms_norm_gain dst"); SEQ_F32(dev, y, "rms_norm_gain y"); SEQ_F32(dev, gain, "rms_norm_gain gain");
@@ -70,7 +98,8 @@ static int rms_norm_gain_impl(cc_device* dev, const cc_view* dst, const cc_view*
     const int64_t rows = y->shape[0], cols = y->shape[1], gn = view_len(gain);
     CC_REQUIRE(dev, gn == 1 || gn == cols, "rms_norm_gain: gain has %lld elements, need 1 or %lld", (long long)gn, (long long)cols);
     if (rows == 0) return CC_OK;
-    rms_norm_gain_kernel<<<(unsigned)((rows + 7) / 8), 256, 0, dev->stream>>>(fptr(dst), fptr(y), fptr(gain), (int)gn, (int)rows, (int)cols, eps, accumulate, mult);
+    if (cols >= 512) rms_norm_gain_wide_kernel<<<(unsigned)rows, RNG_THREADS, 0, dev->stream>>>(fptr(dst), fptr(y), fptr(gain), (int)gn, (int)cols, eps, accumulate, mult);
+    else rms_norm_gain_kernel<<<(unsigned)((rows + 7) / 8), 256, 0, dev->stream>>>(fptr(dst), fptr(y), fptr(gain), (int)gn, (int)rows, (int)cols, eps, accumulate, mult);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
@@ -133,6 +162,33 @@ extern "C" CC_API int cc_glu_inplace(cc_device* dev, const cc_view* gate, const 
     CC_REQUIRE(dev, view_len(up) == n, "glu_inplace: sizes differ");
     if (!n) return CC_OK;
     glu_kernel<<<(unsigned)((n + 255) / 256), 256, 0, dev->stream>>>(fptr(gate), fptr(up), n, act);
+    CC_LAUNCH_CHECK(dev);
+    return CC_OK;
+}
+__global__ void activate_kernel(float* __restrict__ x, int64_t n, int act) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = seq_act(x[i], act);
+}
+extern "C" CC_API int cc_activate_inplace(cc_device* dev, const cc_view* x, int32_t act) {
+    SEQ_ENTER(dev, "activate_inplace");
+    SEQ_F32(dev, x, "activate_inplace x");
+    const int64_t n = view_len(x);
+    if (!n) return CC_OK;
+    activate_kernel<<<(unsigned)((n + 255) / 256), 256, 0, dev->stream>>>(fptr(x), n, act);
+    CC_LAUNCH_CHECK(dev);
+    return CC_OK;
+}
+__global__ void softcap_kernel(float* __restrict__ x, int64_t n, float cap) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+extern "C" CC_API int cc_softcap_inplace(cc_device* dev, const cc_view* x, float cap) {
+    SEQ_ENTER(dev, "softcap_inplace");
+    SEQ_F32(dev, x, "softcap_inplace x");
+    CC_REQUIRE(dev, cap > 0.0f, "softcap_inplace: the cap must be positive");
+    const int64_t n = view_len(x);
+    if (!n) return CC_OK;
+    softcap_kernel<<<(unsigned)((n + 255) / 256), 256, 0, dev->stream>>>(fptr(x), n, cap);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
@@ -300,7 +356,7 @@ extern "C" CC_API int cc_pair_hash_rows_add(cc_device* dev, const cc_view* dst, 
 // one warp per (token, run of hs channels).  in[t'] for t' < 0 comes from the tail: tail row (K-1) + t'.
 // in_bias (or NULL) is added to every input of x as it is read; the tail holds inputs that already carry it (or the zeros before a sequence)
 __global__ void short_conv_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ tail,
-                                  float* __restrict__ y, int T, int C, int K, int hs, int act, int unit, float ueps, float uscale, const float* __restrict__ in_bias) {
+                                  float* __restrict__ y, int T, int C, int K, int hs, int act, int unit, float ueps, float uscale, const float* __restrict__ in_bias, int64_t xrs) {
     const int heads = C / hs;
     const int64_t u = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
@@ -312,7 +368,7 @@ __global__ void short_conv_kernel(const float* __restrict__ x, const float* __re
         float acc = bias ? bias[c] : 0.0f;
         for (int j = 0; j < K; j++) {
             const int ti = t - (K - 1) + j;
-            const float v = ti >= 0 ? (in_bias ? x[(int64_t)ti * C + c] + in_bias[c] : x[(int64_t)ti * C + c]) : tail[(int64_t)(ti + K - 1) * C + c];
+            const float v = ti >= 0 ? (in_bias ? x[ti * xrs + c] + in_bias[c] : x[ti * xrs + c]) : tail[(int64_t)(ti + K - 1) * C + c];
             acc = fmaf(w[(int64_t)c * K + j], v, acc);
         }
         acc = seq_act(acc, act);
@@ -326,22 +382,43 @@ __global__ void short_conv_kernel(const float* __restrict__ x, const float* __re
     }
 }
 // tail <- the last K-1 rows of (tail ++ x); one thread per channel, ascending rows: row j is written after row T + j > j was read
-__global__ void short_conv_tail_kernel(const float* __restrict__ x, float* __restrict__ tail, int T, int C, int K, const float* __restrict__ in_bias) {
-    const int c = blockIdx.x * blockDim.x + threadIdx.x;
-    if (c >= C) return;
-    const float ib = in_bias ? in_bias[c] : 0.0f;
+__device__ __forceinline__ void short_conv_new_tail(const float* x, float* tail, int T, int C, int K, const float* in_bias, int64_t xrs, int c) {
     for (int j = 0; j < K - 1; j++) {
         const int ti = T + j - (K - 1);
-        tail[(int64_t)j * C + c] = ti >= 0 ? (in_bias ? x[(int64_t)ti * C + c] + ib : x[(int64_t)ti * C + c]) : tail[(int64_t)(ti + K - 1) * C + c];
+        tail[(int64_t)j * C + c] = ti >= 0 ? (in_bias ? x[ti * xrs + c] + in_bias[c] : x[ti * xrs + c]) : tail[(int64_t)(ti + K - 1) * C + c];
     }
 }
+__global__ void short_conv_tail_kernel(const float* __restrict__ x, float* tail, int T, int C, int K, const float* __restrict__ in_bias, int64_t xrs) {
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c < C) short_conv_new_tail(x, tail, T, C, K, in_bias, xrs, c);
+}
+// few rows (decoding): one thread per channel walks the rows and then renews its channel's tail -- one launch; the sums are those of
+// short_conv_kernel
+#define SC_FEW_ROWS 8
+__global__ void short_conv_few_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float* tail, float* __restrict__ y, int T, int C,
+                                      int K, int act, const float* __restrict__ in_bias, int64_t xrs) {
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= C) return;
+    for (int t = 0; t < T; t++) {
+        float acc = bias ? bias[c] : 0.0f;
+        for (int j = 0; j < K; j++) {
+            const int ti = t - (K - 1) + j;
+            const float v = ti >= 0 ? (in_bias ? x[ti * xrs + c] + in_bias[c] : x[ti * xrs + c]) : tail[(int64_t)(ti + K - 1) * C + c];
+            acc = fmaf(w[(int64_t)c * K + j], v, acc);
+        }
+        y[(int64_t)t * C + c] = seq_act(acc, act);
+    }
+    short_conv_new_tail(x, tail, T, C, K, in_bias, xrs, c);
+}
 static int short_conv_impl(cc_device* dev, const cc_view* x, const cc_view* w, const cc_view* bias, const cc_view* tail, int32_t act, int32_t head_size, int32_t unit_norm,
-                           float unit_eps, float unit_scale, cc_buf** out, const cc_view* in_bias = nullptr) {
+                           float unit_eps, float unit_scale, cc_buf** out, const cc_view* in_bias = nullptr, int64_t col0 = -1) {
     SEQ_ENTER(dev, "short_conv");
     if (!out) return cc_fail(dev, CC_ERR_ARG, "short_conv: out is NULL");
     SEQ_F32(dev, x, "short_conv x"); SEQ_F32(dev, w, "short_conv w");
-    CC_REQUIRE(dev, x->ndim == 2 && w->ndim == 2 && w->shape[0] == x->shape[1], "short_conv: x must be [T, C] and w [C, K]");
-    const int64_t T = x->shape[0], C = x->shape[1], K = w->shape[1];
+    CC_REQUIRE(dev, x->ndim == 2 && w->ndim == 2 && (col0 < 0 ? w->shape[0] == x->shape[1] : col0 + w->shape[0] <= x->shape[1]),
+               "short_conv: x must be [T, C] (or hold C columns from column %lld on) and w [C, K]", (long long)col0);
+    const int64_t T = x->shape[0], C = w->shape[0], K = w->shape[1], xrs = x->shape[1];
+    const float* xp = fptr(x) + (col0 < 0 ? 0 : col0);
     CC_REQUIRE(dev, K >= 1, "short_conv: no taps");
     if (K > 1) {
         SEQ_F32(dev, tail, "short_conv tail");
@@ -362,12 +439,17 @@ static int short_conv_impl(cc_device* dev, const cc_view* x, const cc_view* w, c
     *out = y;
     if (T == 0) return CC_OK;
     const float* tp = K > 1 ? fptr(tail) : nullptr;
+    if (K > 1 && T <= SC_FEW_ROWS && !unit_norm) {
+        short_conv_few_kernel<<<(unsigned)((C + 127) / 128), 128, 0, dev->stream>>>(xp, fptr(w), bias ? fptr(bias) : nullptr, fptr(tail), (float*)y->base, (int)T, (int)C, (int)K, act, ibp, xrs);
+        CC_LAUNCH_CHECK(dev);
+        return CC_OK;
+    }
     const int64_t units = T * (C / hs);
-    short_conv_kernel<<<(unsigned)((units + 7) / 8), 256, 0, dev->stream>>>(fptr(x), fptr(w), bias ? fptr(bias) : nullptr, tp, (float*)y->base, (int)T, (int)C, (int)K, hs, act, unit_norm,
-                                                                        unit_eps, unit_scale, ibp);
+    short_conv_kernel<<<(unsigned)((units + 7) / 8), 256, 0, dev->stream>>>(xp, fptr(w), bias ? fptr(bias) : nullptr, tp, (float*)y->base, (int)T, (int)C, (int)K, hs, act, unit_norm,
+                                                                        unit_eps, unit_scale, ibp, xrs);
     CC_LAUNCH_CHECK(dev);
     if (K > 1) {
-        short_conv_tail_kernel<<<(unsigned)((C + 127) / 128), 128, 0, dev->stream>>>(fptr(x), fptr(tail), (int)T, (int)C, (int)K, ibp);
+        short_conv_tail_kernel<<<(unsigned)((C + 127) / 128), 128, 0, dev->stream>>>(xp, fptr(tail), (int)T, (int)C, (int)K, ibp, xrs);
         CC_LAUNCH_CHECK(dev);
     }
     return CC_OK;
@@ -383,6 +465,11 @@ extern "C" CC_API int cc_short_conv_biases(cc_device* dev, const cc_view* x, con
 }
 extern "C" CC_API int cc_short_conv_bias(cc_device* dev, const cc_view* x, const cc_view* w, const cc_view* bias, const cc_view* tail, int32_t act, cc_buf** out) {
     return short_conv_impl(dev, x, w, bias, tail, act, 0, 0, 0.0f, 1.0f, out);
+}
+
+extern "C" CC_API int cc_short_conv_cols(cc_device* dev, const cc_view* src, int32_t col0, const cc_view* w, const cc_view* bias, const cc_view* tail, int32_t act, cc_buf** out) {
+    if (dev && col0 < 0) return cc_fail(dev, CC_ERR_ARG, "short_conv_cols: column %d", col0);
+    return short_conv_impl(dev, src, w, bias, tail, act, 0, 0, 0.0f, 1.0f, out, nullptr, col0);
 }
 
 // ---- gated delta rule -------------------------------------------------------------------------------------------------------------
@@ -1093,6 +1180,24 @@ __global__ void group_rms_norm_kernel(float* __restrict__ dst, const float* __re
     float* dr = dst + u * gs;
     for (int c = lane; c < gs; c += 32) dr[c] = xr[c] * inv * wr[c];
 }
+// a wide group: one CTA per (row, group), the order of rms_norm_gain_wide_kernel
+__global__ void __launch_bounds__(RNG_THREADS) group_rms_norm_wide_kernel(float* __restrict__ dst, const float* __restrict__ x, const float* __restrict__ w, int groups, int gs, float eps) {
+    __shared__ float red[RNG_THREADS / 32];
+    const int64_t u = blockIdx.x;
+    const float* xr = x + u * gs;
+    const float* wr = w + (u % groups) * gs;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < gs; c += RNG_THREADS) ss = fmaf(xr[c], xr[c], ss);
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float tot = 0.0f;
+#pragma unroll
+    for (int i = 0; i < RNG_THREADS / 32; i++) tot += red[i];
+    const float inv = 1.0f / sqrtf(tot / (float)gs + eps);
+    float* dr = dst + u * gs;
+    for (int c = threadIdx.x; c < gs; c += RNG_THREADS) dr[c] = xr[c] * inv * wr[c];
+}
 extern "C" CC_API int cc_group_rms_norm(cc_device* dev, const cc_view* dst, const cc_view* x, const cc_view* w, int32_t groups, float eps) {
     SEQ_ENTER(dev, "group_rms_norm");
     SEQ_F32(dev, dst, "group_rms_norm dst"); SEQ_F32(dev, x, "group_rms_norm x"); SEQ_F32(dev, w, "group_rms_norm w");
@@ -1101,7 +1206,8 @@ extern "C" CC_API int cc_group_rms_norm(cc_device* dev, const cc_view* dst, cons
     CC_REQUIRE(dev, groups >= 1 && cols % groups == 0 && view_len(w) == cols, "group_rms_norm: %lld columns, %d groups, %lld weights", (long long)cols, groups, (long long)view_len(w));
     if (rows == 0) return CC_OK;
     const int64_t units = rows * groups;
-    group_rms_norm_kernel<<<(unsigned)((units + 7) / 8), 256, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(w), units, groups, (int)(cols / groups), eps);
+    if (cols / groups >= 512) group_rms_norm_wide_kernel<<<(unsigned)units, RNG_THREADS, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(w), groups, (int)(cols / groups), eps);
+    else group_rms_norm_kernel<<<(unsigned)((units + 7) / 8), 256, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(w), units, groups, (int)(cols / groups), eps);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
@@ -1172,12 +1278,12 @@ extern "C" CC_API int cc_layer_norm(cc_device* dev, const cc_view* dst, const cc
 // the group's size alone (lane- or thread-strided partial sums, the butterfly, then the warps' sums in warp order), and the value is scaled.
 #define GGN_THREADS 256
 __global__ void gated_group_rms_norm_kernel(float* dst, const float* x, const float* __restrict__ gate, const float* __restrict__ w, int64_t n_units,
-                                            int groups, int gs, float eps, int act) {
+                                            int groups, int gs, float eps, int act, int64_t grs) {
     const int64_t u = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     if (u >= n_units) return;
     const float* xr = x + u * gs;
-    const float* gr = gate + u * gs;
+    const float* gr = gate + (u / groups) * grs + (u % groups) * gs;
     const float* wr = w + (u % groups) * gs;
     float* dr = dst + u * gs;
     float ss = 0.0f;
@@ -1187,11 +1293,11 @@ __global__ void gated_group_rms_norm_kernel(float* dst, const float* x, const fl
     for (int c = lane; c < gs; c += 32) dr[c] = dr[c] * inv * wr[c];
 }
 __global__ void __launch_bounds__(GGN_THREADS) gated_group_rms_norm_wide_kernel(float* dst, const float* x, const float* __restrict__ gate,
-                                                                                const float* __restrict__ w, int groups, int gs, float eps, int act) {
+                                                                                const float* __restrict__ w, int groups, int gs, float eps, int act, int64_t grs) {
     __shared__ float red[GGN_THREADS / 32];
     const int64_t u = blockIdx.x;
     const float* xr = x + u * gs;
-    const float* gr = gate + u * gs;
+    const float* gr = gate + (u / groups) * grs + (u % groups) * gs;
     const float* wr = w + (u % groups) * gs;
     float* dr = dst + u * gs;
     float ss = 0.0f;
@@ -1208,17 +1314,18 @@ __global__ void __launch_bounds__(GGN_THREADS) gated_group_rms_norm_wide_kernel(
 extern "C" CC_API int cc_gated_group_rms_norm(cc_device* dev, const cc_view* dst, const cc_view* x, const cc_view* gate, const cc_view* w, int32_t groups, float eps,
                                               int32_t gate_act) {
     SEQ_ENTER(dev, "gated_group_rms_norm");
-    SEQ_F32(dev, dst, "gated_group_rms_norm dst"); SEQ_F32(dev, x, "gated_group_rms_norm x"); SEQ_F32(dev, gate, "gated_group_rms_norm gate"); SEQ_F32(dev, w, "gated_group_rms_norm w");
-    CC_REQUIRE(dev, x->ndim == 2 && dst->ndim == 2 && dst->shape[0] == x->shape[0] && dst->shape[1] == x->shape[1] && view_len(gate) == view_len(x),
+    SEQ_F32(dev, dst, "gated_group_rms_norm dst"); SEQ_F32(dev, x, "gated_group_rms_norm x"); SEQ_ROWS(dev, gate, "gated_group_rms_norm gate"); SEQ_F32(dev, w, "gated_group_rms_norm w");
+    CC_REQUIRE(dev, x->ndim == 2 && dst->ndim == 2 && dst->shape[0] == x->shape[0] && dst->shape[1] == x->shape[1] && gate->shape[0] == x->shape[0] && gate->shape[1] == x->shape[1],
                "gated_group_rms_norm: dst, x and gate must be [rows, cols]");
+    const int64_t grs = gate->strides[0];
     const int64_t rows = x->shape[0], cols = x->shape[1];
     CC_REQUIRE(dev, groups >= 1 && cols % groups == 0 && view_len(w) == cols, "gated_group_rms_norm: %lld columns, %d groups, %lld weights", (long long)cols, groups,
                (long long)view_len(w));
     if (rows == 0) return CC_OK;
     const int64_t units = rows * groups;
     const int gs = (int)(cols / groups);
-    if (gs >= 512) gated_group_rms_norm_wide_kernel<<<(unsigned)units, GGN_THREADS, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(gate), fptr(w), groups, gs, eps, gate_act);
-    else gated_group_rms_norm_kernel<<<(unsigned)((units + 7) / 8), 256, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(gate), fptr(w), units, groups, gs, eps, gate_act);
+    if (gs >= 512) gated_group_rms_norm_wide_kernel<<<(unsigned)units, GGN_THREADS, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(gate), fptr(w), groups, gs, eps, gate_act, grs);
+    else gated_group_rms_norm_kernel<<<(unsigned)((units + 7) / 8), 256, 0, dev->stream>>>(fptr(dst), fptr(x), fptr(gate), fptr(w), units, groups, gs, eps, gate_act, grs);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
@@ -1394,13 +1501,19 @@ extern "C" CC_API int cc_qk_prepare_append(cc_device* dev, const cc_view* q, con
 
 // ---- latent key/value cache ------------------------------------------------------------------------------------------------------------------
 // one warp per token: the first `rank` columns are RMS-normalised and weighted, the pairs of the next columns rotated, the rest copied
-__global__ void latent_ring_append_kernel(float* __restrict__ ring, const float* __restrict__ ckv, const float* __restrict__ nw, const float* __restrict__ freq, float eps,
-                                          float mag, int64_t pos0, int ring_rows, int T, int rank, int rest, int half) {
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (t >= T) return;
-    const int cols = rank + rest;
-    const float* src = ckv + (int64_t)t * cols;
-    float* dst = ring + ((pos0 + t) % ring_rows) * cols;
+struct LatAppend {
+    float* ring;                  // NULL: nothing to append
+    const float *ckv, *nw, *freq; // row t of the raw rows at ckv + t * rs
+    int64_t rs, pos0;
+    int ring_rows, rank, rest, half;
+    float eps, mag;
+};
+__device__ __forceinline__ void latent_append_row(const LatAppend& a, int t, int lane) {
+    const int rank = a.rank, cols = a.rank + a.rest, half = a.half;
+    const int64_t pos0 = a.pos0;
+    const float *nw = a.nw, *freq = a.freq, *src = a.ckv + t * a.rs;
+    const float eps = a.eps, mag = a.mag;
+    float* dst = a.ring + ((pos0 + t) % a.ring_rows) * cols;
     float ss = 0.0f;
     for (int c = lane; c < rank; c += 32) ss = fmaf(src[c], src[c], ss);
     ss = warp_sum(ss);
@@ -1412,6 +1525,10 @@ __global__ void latent_ring_append_kernel(float* __restrict__ ring, const float*
         dst[rank + 2 * i] = ou; dst[rank + 2 * i + 1] = ov;
     }
     for (int c = rank + 2 * half + lane; c < cols; c += 32) dst[c] = src[c];
+}
+__global__ void latent_ring_append_kernel(LatAppend a, int T) {
+    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (t < T) latent_append_row(a, t, threadIdx.x & 31);
 }
 extern "C" CC_API int cc_latent_ring_append(cc_device* dev, const cc_view* ring, const cc_view* ckv, const cc_view* norm_w, float eps, int32_t rank, const cc_view* freq,
                                             float mag, int64_t pos0) {
@@ -1425,45 +1542,58 @@ extern "C" CC_API int cc_latent_ring_append(cc_device* dev, const cc_view* ring,
                (long long)half, (long long)cols);
     CC_REQUIRE(dev, T <= ring->shape[0], "latent_ring_append: %lld tokens do not fit a ring of %lld", (long long)T, (long long)ring->shape[0]);
     if (T == 0) return CC_OK;
-    latent_ring_append_kernel<<<(unsigned)((T + 7) / 8), 256, 0, dev->stream>>>(fptr(ring), fptr(ckv), norm_w ? fptr(norm_w) : nullptr, freq ? fptr(freq) : nullptr, eps, mag, pos0,
-                                                                                  (int)ring->shape[0], (int)T, rank, (int)(cols - rank), (int)half);
+    const LatAppend a = {fptr(ring), fptr(ckv), norm_w ? fptr(norm_w) : nullptr, freq ? fptr(freq) : nullptr, cols, pos0, (int)ring->shape[0], rank, (int)(cols - rank), (int)half, eps, mag};
+    latent_ring_append_kernel<<<(unsigned)((T + 7) / 8), 256, 0, dev->stream>>>(a, (int)T);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
 
 // ---- per-head products: the up-projections of a latent cache, folded into the query and applied to the attention result ---------------------
 #define HP_TOK 8
+struct HpArgs {
+    const float *x, *W;           // token t's row at x + t * xrs, head h's inputs at + h * (n_in + rest)
+    float* out;
+    int64_t xrs, grs, pos0;
+    const float *freq, *gate;     // gate (rest == 0 only): output (t, h, v) is multiplied by sigmoid(gate[t * grs + h * n_out + v]); NULL: not gated
+    int T, H, n_in, rest, n_out, half;
+    float mag;
+    LatAppend app;                // app.ring != NULL: the grid has one more z plane, whose CTAs of head 0 write the tokens' cache rows
+};
 // grid (ceil(T / 8), H, ceil(n_out / 4)): the CTA stages 8 tokens' x[t, h, :n_in]; a warp owns one output coordinate for those tokens:
 // lane-strided partial sums over n_in, then the butterfly -- one order per output, whatever T is.  W: [H * n_out, n_in], rows read
 // contiguously.  The `rest` columns behind a head's n_in inputs are copied behind its n_out outputs.
-__global__ void __launch_bounds__(128) head_project_kernel(const float* __restrict__ x, const float* __restrict__ W, float* __restrict__ out, int T, int H, int n_in, int rest,
-                                                           int n_out, const float* __restrict__ freq, int half, float mag, int64_t pos0) {
+__global__ void __launch_bounds__(128) head_project_kernel(HpArgs a) {
     extern __shared__ float hp_sm[];
-    const int t0 = blockIdx.x * HP_TOK, h = blockIdx.y;
+    const int t0 = blockIdx.x * HP_TOK, h = blockIdx.y, T = a.T, H = a.H, n_in = a.n_in, rest = a.rest, n_out = a.n_out, half = a.half;
+    if (a.app.ring && blockIdx.z == gridDim.z - 1) {
+        if (h == 0)
+            for (int tt = threadIdx.x >> 5; tt < HP_TOK && t0 + tt < T; tt += 4) latent_append_row(a.app, t0 + tt, threadIdx.x & 31);
+        return;
+    }
     const int xs = n_in + rest, os = n_out + rest;
     for (int i = threadIdx.x; i < HP_TOK * n_in; i += 128) {
         const int tt = i / n_in, d = i - tt * n_in;
-        hp_sm[i] = t0 + tt < T ? x[((int64_t)(t0 + tt) * H + h) * xs + d] : 0.0f;
+        hp_sm[i] = t0 + tt < T ? a.x[(t0 + tt) * a.xrs + h * xs + d] : 0.0f;
     }
     if (blockIdx.z == 0) {
         // the carried columns: the first 2 * half of them are rotated on the way when a frequency table is given
         for (int i = threadIdx.x; i < HP_TOK * half; i += 128) {
             const int tt = i / half, p = i - tt * half;
             if (t0 + tt >= T) continue;
-            const float* src = x + ((int64_t)(t0 + tt) * H + h) * xs + n_in + 2 * p;
-            float* dst = out + ((int64_t)(t0 + tt) * H + h) * os + n_out + 2 * p;
-            rotate_pair(src[0], src[1], (float)(pos0 + t0 + tt), freq[p], mag, dst[0], dst[1]);
+            const float* src = a.x + (t0 + tt) * a.xrs + h * xs + n_in + 2 * p;
+            float* dst = a.out + ((int64_t)(t0 + tt) * H + h) * os + n_out + 2 * p;
+            rotate_pair(src[0], src[1], (float)(a.pos0 + t0 + tt), a.freq[p], a.mag, dst[0], dst[1]);
         }
         const int plain = rest - 2 * half;
         for (int i = threadIdx.x; i < HP_TOK * plain; i += 128) {
             const int tt = i / plain, j = 2 * half + (i - tt * plain);
-            if (t0 + tt < T) out[((int64_t)(t0 + tt) * H + h) * os + n_out + j] = x[((int64_t)(t0 + tt) * H + h) * xs + n_in + j];
+            if (t0 + tt < T) a.out[((int64_t)(t0 + tt) * H + h) * os + n_out + j] = a.x[(t0 + tt) * a.xrs + h * xs + n_in + j];
         }
     }
     __syncthreads();
     const int v = blockIdx.z * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (v >= n_out) return;
-    const float* wp = W + ((int64_t)h * n_out + v) * n_in;
+    const float* wp = a.W + ((int64_t)h * n_out + v) * n_in;
     float acc[HP_TOK];
 #pragma unroll
     for (int tt = 0; tt < HP_TOK; tt++) acc[tt] = 0.0f;
@@ -1474,9 +1604,19 @@ __global__ void __launch_bounds__(128) head_project_kernel(const float* __restri
     }
 #pragma unroll
     for (int tt = 0; tt < HP_TOK; tt++) {
-        const float sum = warp_sum(acc[tt]);
-        if (lane == 0 && t0 + tt < T) out[((int64_t)(t0 + tt) * H + h) * os + v] = sum;
+        float sum = warp_sum(acc[tt]);
+        if (lane != 0 || t0 + tt >= T) continue;
+        if (a.gate) sum *= seq_sigmoid(a.gate[(t0 + tt) * a.grs + h * n_out + v]);
+        a.out[((int64_t)(t0 + tt) * H + h) * os + v] = sum;
     }
+}
+static int head_project_few(cc_device* dev, const HpArgs& a) {
+    const size_t smem = (size_t)HP_TOK * a.n_in * 4;
+    CC_REQUIRE(dev, smem <= 160 * 1024, "head_project: %d inputs per head do not fit shared memory", a.n_in);
+    if (smem > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(head_project_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    head_project_kernel<<<dim3((unsigned)((a.T + HP_TOK - 1) / HP_TOK), (unsigned)a.H, (unsigned)((a.n_out + 3) / 4 + (a.app.ring ? 1 : 0))), 128, smem, dev->stream>>>(a);
+    CC_LAUNCH_CHECK(dev);
+    return CC_OK;
 }
 // many rows and nothing carried: a 64 x 64 output tile of one head per CTA, 16-deep slices of the inputs through shared memory, 4 x 4 outputs
 // per thread, every sum over n_in in ascending order inside one thread.  grid (ceil(n_out / 64), ceil(T / 64), H)
@@ -1549,11 +1689,57 @@ extern "C" CC_API int cc_head_project(cc_device* dev, const cc_view* x, const cc
         CC_LAUNCH_CHECK(dev);
         return CC_OK;
     }
-    if (smem > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(head_project_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    head_project_kernel<<<dim3((unsigned)((T + HP_TOK - 1) / HP_TOK), (unsigned)n_heads, (unsigned)((n_out + 3) / 4)), 128, smem, dev->stream>>>(
-        fptr(x), fptr(w), (float*)o->base, (int)T, n_heads, (int)n_in, rest, (int)n_out, freq ? fptr(freq) : nullptr, freq ? (int)view_len(freq) : 0, mag, pos0);
-    CC_LAUNCH_CHECK(dev);
-    return CC_OK;
+    HpArgs a{};
+    a.x = fptr(x); a.W = fptr(w); a.out = (float*)o->base; a.xrs = x->shape[1]; a.pos0 = pos0; a.freq = freq ? fptr(freq) : nullptr; a.half = freq ? (int)view_len(freq) : 0; a.mag = mag;
+    a.T = (int)T; a.H = n_heads; a.n_in = (int)n_in; a.rest = rest; a.n_out = (int)n_out;
+    return head_project_few(dev, a);
+}
+extern "C" CC_API int cc_head_project_gated(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, cc_buf** out) {
+    SEQ_ENTER(dev, "head_project_gated");
+    if (!out) return cc_fail(dev, CC_ERR_ARG, "head_project_gated: out is NULL");
+    SEQ_F32(dev, x, "head_project_gated x"); SEQ_F32(dev, w, "head_project_gated w"); SEQ_ROWS(dev, gate_src, "head_project_gated gate");
+    CC_REQUIRE(dev, x->ndim == 2 && w->ndim == 2 && n_heads > 0 && w->shape[0] % n_heads == 0 && x->shape[1] == (int64_t)n_heads * w->shape[1],
+               "head_project_gated: x must be [T, heads * n_in] and w [heads * n_out, n_in]");
+    const int64_t T = x->shape[0];
+    CC_REQUIRE(dev, gate_src->shape[0] == T && gate_col0 >= 0 && gate_col0 + w->shape[0] <= gate_src->shape[1], "head_project_gated: the gate needs %lld columns from column %d on",
+               (long long)w->shape[0], gate_col0);
+    cc_buf* o = nullptr;
+    int rc = cc_new_activation(dev, T * w->shape[0], CC_F32, false, &o);
+    if (rc) return rc;
+    *out = o;
+    if (T == 0) return CC_OK;
+    HpArgs a{};
+    a.x = fptr(x); a.W = fptr(w); a.out = (float*)o->base; a.xrs = x->shape[1]; a.gate = fptr(gate_src) + gate_col0; a.grs = gate_src->strides[0]; a.mag = 1.0f;
+    a.T = (int)T; a.H = n_heads; a.n_in = (int)w->shape[1]; a.n_out = (int)(w->shape[0] / n_heads);
+    return head_project_few(dev, a);
+}
+extern "C" CC_API int cc_latent_query_append(cc_device* dev, const cc_view* q_src, int32_t q_col0, const cc_view* uk_t, int32_t n_heads, int32_t rest, const cc_view* freq, float mag,
+                                             int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps, cc_buf** out) {
+    SEQ_ENTER(dev, "latent_query_append");
+    if (!out) return cc_fail(dev, CC_ERR_ARG, "latent_query_append: out is NULL");
+    SEQ_ROWS(dev, q_src, "latent_query_append q"); SEQ_F32(dev, uk_t, "latent_query_append uk_t");
+    CC_REQUIRE(dev, uk_t->ndim == 2 && n_heads > 0 && rest >= 0 && uk_t->shape[0] % n_heads == 0 && pos0 >= 0, "latent_query_append: bad arguments");
+    const int64_t T = q_src->shape[0], dim = uk_t->shape[1], rank = uk_t->shape[0] / n_heads;
+    CC_REQUIRE(dev, q_col0 >= 0 && q_col0 + n_heads * (dim + rest) <= q_src->shape[1], "latent_query_append: the queries need %lld columns from column %d on",
+               (long long)(n_heads * (dim + rest)), q_col0);
+    if (freq) { SEQ_F32(dev, freq, "latent_query_append freq"); CC_REQUIRE(dev, 2 * view_len(freq) <= rest, "latent_query_append: more rotated pairs than carried columns"); }
+    HpArgs a{};
+    if (kv_src) {
+        SEQ_ROWS(dev, kv_src, "latent_query_append kv"); SEQ_F32(dev, ring, "latent_query_append ring");
+        if (norm_w) { SEQ_F32(dev, norm_w, "latent_query_append norm_w"); CC_REQUIRE(dev, view_len(norm_w) == rank, "latent_query_append: norm_w must have %lld elements", (long long)rank); }
+        CC_REQUIRE(dev, ring->ndim == 2 && ring->shape[1] == rank + rest && T <= ring->shape[0] && kv_src->shape[0] == T && kv_col0 >= 0 && kv_col0 + rank + rest <= kv_src->shape[1],
+                   "latent_query_append: ring rows have rank + rest columns and so have the raw rows from column %d on", kv_col0);
+        a.app = {fptr(ring), fptr(kv_src) + kv_col0, norm_w ? fptr(norm_w) : nullptr, freq ? fptr(freq) : nullptr, kv_src->strides[0], pos0, (int)ring->shape[0], (int)rank, rest,
+                 freq ? (int)view_len(freq) : 0, eps, mag};
+    }
+    cc_buf* o = nullptr;
+    int rc = cc_new_activation(dev, T * n_heads * (rank + rest), CC_F32, false, &o);
+    if (rc) return rc;
+    *out = o;
+    if (T == 0) return CC_OK;
+    a.x = fptr(q_src) + q_col0; a.W = fptr(uk_t); a.out = (float*)o->base; a.xrs = q_src->strides[0]; a.pos0 = pos0; a.freq = freq ? fptr(freq) : nullptr;
+    a.half = freq ? (int)view_len(freq) : 0; a.mag = mag; a.T = (int)T; a.H = n_heads; a.n_in = (int)dim; a.rest = rest; a.n_out = (int)rank;
+    return head_project_few(dev, a);
 }
 
 // out[j, h] = [ a[j, h, :dim] | shared[j, col0 : col0 + rest] ]: every head's part followed by the columns all heads share.  One thread per element.

@@ -28,11 +28,19 @@ static inline float* lptr(const cc_view* v) { return (float*)v->buf->plane[0]; }
 __device__ __forceinline__ float lin_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float lin_softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 
+// the state-space step of a (token, head): {exp(-exp(a_log) d), d}, d = softplus(dt + dt_bias)
+__device__ __forceinline__ float2 ss_step(float dt, float dt_bias, float a_log) {
+    const float d = lin_softplus(dt + dt_bias);
+    return make_float2(expf(-expf(a_log) * d), d);
+}
+
 // ---- the recurrence ------------------------------------------------------------------------------------------------------------------------
 struct LrArgs {
     const float *q, *k, *v;       // q, k: row t at + t * rs, the head group's dk numbers at + g * dk; v: row t at + t * v_rs, head h's at + h * v_hs
     const float* adec;            // [T, H * dk] decay per key channel, or NULL
     const float* sc;              // [T, H, 2] = {decay, weight of the outer product} per (token, head), or NULL (1, 1)
+    const float *dt, *dt_bias, *a_log;   // sc is NULL and dt is not: {decay, weight} are taken from the raw step sizes (row t at dt + t * dt_rs) while a block is staged
+    int64_t dt_rs;
     const float* hdec;            // [H] one decay per head for every token, or NULL (1); read only when sc is NULL
     float wgt;                    // weight of the outer product when sc is NULL
     const float* skip;            // [H] or NULL: out += skip[h] * v
@@ -93,6 +101,7 @@ __global__ void __launch_bounds__(DK > 0 ? LR_COLS * SPLIT : LR_GENERIC_THREADS)
         for (int idx = threadIdx.x; idx < 2 * n_rows; idx += THREADS)
             for (int i = dk; i < dk4; i++) lr_sm[(idx / n_rows) * stage_floats + (idx % n_rows) * dk4 + i] = 0.0f;
     const float skip = a.skip ? a.skip[h] : 0.0f;
+    const bool staged = a.sc || a.dt;                       // decay and weight per token come with the block
     const float head_dec = a.hdec ? a.hdec[h] : 1.0f;
     // a thread's first piece of a block of tokens, and how far the next one is: item idx = threadIdx.x + n THREADS is token idx / per,
     // piece idx % per of the block; walked without divisions
@@ -120,6 +129,8 @@ __global__ void __launch_bounds__(DK > 0 ? LR_COLS * SPLIT : LR_GENERIC_THREADS)
         float* ssc = base + n_rows * dk4;
         if (a.sc)
             for (int idx = threadIdx.x; idx < nt * 2; idx += THREADS) lr_cp4(ssc + idx, a.sc + ((int64_t)(tb + (idx >> 1)) * a.H + h) * 2 + (idx & 1));
+        else if (a.dt && threadIdx.x < nt)
+            *(float2*)(ssc + 2 * threadIdx.x) = ss_step(a.dt[(int64_t)(tb + threadIdx.x) * a.dt_rs + h], a.dt_bias[h], a.a_log[h]);
         // the block's values of the CTA's columns: [token][column]
         float* sv = ssc + 2 * LR_TB;
         for (int idx = threadIdx.x; idx < nt * COLS; idx += THREADS) {
@@ -146,7 +157,7 @@ __global__ void __launch_bounds__(DK > 0 ? LR_COLS * SPLIT : LR_GENERIC_THREADS)
             const float* kt = base + tt * dk4 + 4 * part;
             const float* qt = base + (LR_TB + tt) * dk4 + 4 * part;
             const float* dt = base + (2 * LR_TB + tt) * dk4 + 4 * part;
-            const float dec = a.sc ? ssc[tt * 2] : head_dec, wgt = a.sc ? ssc[tt * 2 + 1] : a.wgt;
+            const float dec = staged ? ssc[tt * 2] : head_dec, wgt = staged ? ssc[tt * 2 + 1] : a.wgt;
             const float vj = ones ? 1.0f : sv[tt * COLS];
             const float u = wgt * vj;
             float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
@@ -391,17 +402,16 @@ extern "C" CC_API int cc_retention(cc_device* dev, const cc_view* q, const cc_vi
 }
 
 // ---- selective state-space scan ------------------------------------------------------------------------------------------------------------------
-// sc[(t * H + h) * 2] = {exp(-exp(a_log) d), d}, d = softplus(dt + dt_bias)
-__global__ void ss_steps_kernel(const float* __restrict__ dt, const float* __restrict__ dt_bias, const float* __restrict__ a_log, float* __restrict__ sc, int64_t n, int H) {
+// sc[(t * H + h) * 2] = ss_step of the token and head
+__global__ void ss_steps_kernel(const float* __restrict__ dt, const float* __restrict__ dt_bias, const float* __restrict__ a_log, float* __restrict__ sc, int64_t n, int H,
+                                int64_t dt_rs) {
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const int h = (int)(i % H);
-    const float d = lin_softplus(dt[i] + dt_bias[h]);
-    sc[i * 2] = expf(-expf(a_log[h]) * d);
-    sc[i * 2 + 1] = d;
+    *(float2*)(sc + i * 2) = ss_step(dt[(i / H) * dt_rs + h], dt_bias[h], a_log[h]);
 }
-extern "C" CC_API int cc_state_space_scan(cc_device* dev, const cc_view* xbc, const cc_view* dt, const cc_view* dt_bias, const cc_view* a_log, const cc_view* d_skip,
-                                          const cc_view* state, int32_t H, int32_t G, int32_t N, int32_t P, cc_buf** out) {
+static int state_space_scan_impl(cc_device* dev, const cc_view* xbc, const cc_view* dt, int64_t dt_col0, const cc_view* dt_bias, const cc_view* a_log, const cc_view* d_skip,
+                                 const cc_view* state, int32_t H, int32_t G, int32_t N, int32_t P, cc_buf** out) {
     LIN_ENTER(dev, "state_space_scan");
     if (!out) return cc_fail(dev, CC_ERR_ARG, "state_space_scan: out is NULL");
     LIN_F32(dev, xbc, "state_space_scan xbc"); LIN_F32(dev, dt, "state_space_scan dt"); LIN_F32(dev, dt_bias, "state_space_scan dt_bias");
@@ -409,27 +419,43 @@ extern "C" CC_API int cc_state_space_scan(cc_device* dev, const cc_view* xbc, co
     if (d_skip) LIN_F32(dev, d_skip, "state_space_scan d_skip");
     CC_REQUIRE(dev, H > 0 && G > 0 && H % G == 0 && N > 0 && P > 0 && xbc->ndim == 2, "state_space_scan: bad head counts / sizes");
     const int64_t T = xbc->shape[0], row = (int64_t)H * P + 2 * (int64_t)G * N;
-    CC_REQUIRE(dev, xbc->shape[1] == row && view_len(dt) == T * H && view_len(dt_bias) == H && view_len(a_log) == H && (!d_skip || view_len(d_skip) == H) &&
-                        view_len(state) == (int64_t)H * N * P,
+    CC_REQUIRE(dev, xbc->shape[1] == row && (dt_col0 < 0 ? view_len(dt) == T * H : dt->ndim == 2 && dt->shape[0] == T && dt_col0 + H <= dt->shape[1]) && view_len(dt_bias) == H &&
+                        view_len(a_log) == H && (!d_skip || view_len(d_skip) == H) && view_len(state) == (int64_t)H * N * P,
                "state_space_scan: operand sizes do not fit T=%lld heads=%d groups=%d state=%d head_dim=%d", (long long)T, H, G, N, P);
     cc_buf* o = nullptr;
     int rc = cc_new_activation(dev, T * H * P, CC_F32, false, &o);
     if (rc) return rc;
     *out = o;
     if (T == 0) return CC_OK;
-    void* tmp = nullptr; size_t cls = 0;
-    rc = cc_pool_alloc(dev, (size_t)T * H * 2 * 4, &tmp, &cls);
-    if (rc) return rc;
-    ss_steps_kernel<<<(unsigned)((T * H + 255) / 256), 256, 0, dev->stream>>>(lptr(dt), lptr(dt_bias), lptr(a_log), (float*)tmp, T * H, H);
-    dev->launches++;
     LrArgs a{};
     const float* base = lptr(xbc);
-    a.v = base; a.k = base + (int64_t)H * P; a.q = base + (int64_t)H * P + (int64_t)G * N; a.adec = nullptr; a.sc = (const float*)tmp;
+    const float* dtp = lptr(dt) + (dt_col0 < 0 ? 0 : dt_col0);
+    const int64_t dt_rs = dt_col0 < 0 ? H : dt->shape[1];
+    a.v = base; a.k = base + (int64_t)H * P; a.q = base + (int64_t)H * P + (int64_t)G * N; a.adec = nullptr;
     a.skip = d_skip ? lptr(d_skip) : nullptr; a.state = lptr(state); a.out = (float*)o->base;
     a.T = (int)T; a.H = H; a.G = G; a.dk = N; a.dv = P; a.q_rs = a.k_rs = a.v_rs = (int)row; a.v_hs = P; a.q_scale = 1.0f; a.wgt = 1.0f;
+    void* tmp = nullptr; size_t cls = 0;
+    if (T <= LR_TB) {                      // one block of tokens: the kernel takes the steps itself, the same numbers
+        a.dt = dtp; a.dt_rs = dt_rs; a.dt_bias = lptr(dt_bias); a.a_log = lptr(a_log);
+    } else {
+        rc = cc_pool_alloc(dev, (size_t)T * H * 2 * 4, &tmp, &cls);
+        if (rc) return rc;
+        ss_steps_kernel<<<(unsigned)((T * H + 255) / 256), 256, 0, dev->stream>>>(dtp, lptr(dt_bias), lptr(a_log), (float*)tmp, T * H, H, dt_rs);
+        dev->launches++;
+        a.sc = (const float*)tmp;
+    }
     rc = lr_launch(dev, a, "state_space_scan");
-    cc_pool_free(dev, tmp, cls);
+    if (tmp) cc_pool_free(dev, tmp, cls);
     if (rc) return rc;
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
+}
+extern "C" CC_API int cc_state_space_scan(cc_device* dev, const cc_view* xbc, const cc_view* dt, const cc_view* dt_bias, const cc_view* a_log, const cc_view* d_skip,
+                                          const cc_view* state, int32_t H, int32_t G, int32_t N, int32_t P, cc_buf** out) {
+    return state_space_scan_impl(dev, xbc, dt, -1, dt_bias, a_log, d_skip, state, H, G, N, P, out);
+}
+extern "C" CC_API int cc_state_space_scan_cols(cc_device* dev, const cc_view* xbc, const cc_view* dt_src, int32_t dt_col0, const cc_view* dt_bias, const cc_view* a_log,
+                                               const cc_view* d_skip, const cc_view* state, int32_t H, int32_t G, int32_t N, int32_t P, cc_buf** out) {
+    if (dev && dt_col0 < 0) return cc_fail(dev, CC_ERR_ARG, "state_space_scan_cols: column %d", dt_col0);
+    return state_space_scan_impl(dev, xbc, dt_src, dt_col0, dt_bias, a_log, d_skip, state, H, G, N, P, out);
 }

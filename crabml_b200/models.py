@@ -70,3 +70,11 @@ def _load_lifesun(path, device, dtype="bfloat16", chunk=0, max_tokens=0, **_):
 
 
 register("Lifesun", _load_lifesun)
+
+
+def _load_papunex(path, device, dtype="bfloat16", chunk=0, max_tokens=0, **_):
+    from . import papunex
+    return papunex.load(path, device, dtype, chunk, max_tokens)
+
+
+register("Papunex", _load_papunex)

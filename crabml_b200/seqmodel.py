@@ -108,10 +108,48 @@ class Uploader:
         return self._mat_from(None, np.asarray(a)) if name in self.bf16_names else self._mat_from(np.asarray(a, np.float32), None)
 
     def stack(self, names) -> CudaTensor:
-        """the named matrices one under the other (expert-major stacks)"""
-        if all(n in self.bf16_names for n in names):
-            return self._mat_from(None, np.concatenate([np.asarray(self.weights[n]) for n in names], 0))
-        return self._mat_from(np.concatenate([self.f32(n) for n in names], 0), None)
+        """the named matrices one under the other (expert-major stacks).  An entry may be (name, cut): cut(array) is stacked instead of the
+        array; it slices or zero-pads and must not depend on the values (bfloat16 tensors reach it as bit patterns)."""
+        names = [n if isinstance(n, tuple) else (n, lambda a: a) for n in names]
+        if all(n in self.bf16_names for n, _ in names):
+            return self._mat_from(None, np.concatenate([cut(np.asarray(self.weights[n])) for n, cut in names], 0))
+        return self._mat_from(np.concatenate([cut(self.f32(n)) for n, cut in names], 0), None)
+
+    # ---- what mixers of several families upload (csrc/host/mixers.hpp) ------------------------------------------------------------------
+    def latent_projections(self, p, heads, dim, kv_rank) -> dict:
+        """p: '<layer>.mix.'.  uk, uv for the dense products of a pass of many rows; for a pass of few rows, which folds the up-projections
+        into the 32-bit scores and sums, F32 copies, the key one transposed head by head; the sink where the file has one"""
+        uk = self.f32(p + "uk").reshape(heads, dim, kv_rank)
+        t = {"uk": self.mat(p + "uk"), "uv": self.mat(p + "uv"),
+             "uk_t": self.table(np.ascontiguousarray(uk.transpose(0, 2, 1)).reshape(heads * kv_rank, dim))}
+        t["uv_f32"] = t["uv"] if self.dtype == "float32" else self.mat32(p + "uv")
+        if p + "sink" in self.weights:
+            t["sink"] = self.vec(p + "sink")
+        return t
+
+    def state_space(self, p) -> dict:
+        """p: '<layer>.mix.'"""
+        return {"in": self.mat(p + "in"), "conv": self.mat32(p + "conv"), "conv_bias": self.vec(p + "conv.b"), "dt_bias": self.vec(p + "dt_bias"), "a_log": self.vec(p + "A_log"),
+                "d_skip": self.vec(p + "D"), "s_norm": self.vec(p + "norm"), "s_o": self.mat(p + "o")}
+
+
+# ---- the state-space mixer's entry of a config.json, shared by the families that have one ---------------------------------------------------
+STATE_SPACE_FIELDS = {"heads": "s_heads", "vdim": "s_vdim", "state": "s_state", "groups": "s_groups", "conv": "s_conv", "norm_groups": "s_norm_groups"}
+
+
+def parse_state_space(m: dict, at: str) -> dict:
+    out = {k: int(m[k]) for k in ("heads", "vdim", "state", "conv")}
+    out["groups"], out["norm_groups"] = int(m.get("groups", 1)), int(m.get("norm_groups", 1))
+    if out["heads"] % out["groups"] or (out["heads"] * out["vdim"]) % out["norm_groups"]:
+        raise TensorError(f"{at}: groups / norm_groups do not divide the heads / the inner width")
+    return out
+
+
+def state_space_tensors(m: dict, p: str, width: int) -> dict:
+    """name -> shape of the mixer's tensors; p: '<layer>.mix.'"""
+    inner, bc = m["heads"] * m["vdim"], 2 * m["groups"] * m["state"]
+    return {p + "in": [2 * inner + bc + m["heads"], width], p + "conv": [inner + bc, m["conv"]], p + "conv.b": [inner + bc], p + "dt_bias": [m["heads"]], p + "A_log": [m["heads"]],
+            p + "D": [m["heads"]], p + "norm": [inner], p + "o": [width, inner]}
 
 
 def handle_of(t: CudaTensor):

@@ -130,9 +130,10 @@ def window_attention_sink(q, kring, vring, pos0, n_heads, n_kv, dk, dv, window, 
     return _new(q.device, h, [q.shape()[0], n_heads * dv])
 
 
-def moe_route_ex(x, router_w, correction, top, n_groups=1, keep_groups=1, score=capi.ROUTE_SOFTMAX, group_top=1, renormalise=False, renorm_eps=0.0):
+def moe_route_ex(x, router_w, correction, top, n_groups=1, keep_groups=1, score=capi.ROUTE_SOFTMAX, group_top=1, renormalise=False, renorm_eps=0.0,
+                 scale=1.0):
     hi, hw = C.c_void_p(), C.c_void_p()
-    rp = capi.cc_route_params(int(score), int(top), int(n_groups), int(keep_groups), int(group_top), int(renormalise), float(renorm_eps))
+    rp = capi.cc_route_params(int(score), int(top), int(n_groups), int(keep_groups), int(group_top), int(renormalise), float(renorm_eps), float(scale))
     x.device.check(x.device.lib.cc_moe_route_ex(x.device.handle, _v(x), _v(router_w), _v(correction), C.byref(rp), C.byref(hi), C.byref(hw)))
     T = x.shape()[0]
     return _new(x.device, hi, [T, top]), _new(x.device, hw, [T, top])
@@ -287,3 +288,65 @@ def short_conv_biases(x, w, in_bias, bias, tail, act=capi.ACT_NONE):
     h = C.c_void_p()
     x.device.check(x.device.lib.cc_short_conv_biases(x.device.handle, _v(x), _v(w), _v(in_bias), _v(bias), _v(tail), int(act), C.byref(h)))
     return _new(x.device, h, x.shape())
+
+
+def activate_inplace(x, act):
+    x.device.check(x.device.lib.cc_activate_inplace(x.device.handle, _v(x), int(act)))
+    return x
+
+
+def softcap_inplace(x, cap):
+    x.device.check(x.device.lib.cc_softcap_inplace(x.device.handle, _v(x), float(cap)))
+    return x
+
+
+def short_conv_cols(src, col0, w, bias, tail, act=capi.ACT_SILU):
+    """the convolution over the columns col0 .. col0 + C of a wider matrix"""
+    h = C.c_void_p()
+    src.device.check(src.device.lib.cc_short_conv_cols(src.device.handle, _v(src), int(col0), _v(w), _v(bias), _v(tail), int(act), C.byref(h)))
+    return _new(src.device, h, [src.shape()[0], w.shape()[0]])
+
+
+def state_space_scan_cols(xbc, dt_src, dt_col0, dt_bias, a_log, d_skip, state, n_heads, n_groups, n_state, head_dim):
+    """state_space_scan with the raw step sizes in columns of a wider matrix"""
+    h = C.c_void_p()
+    xbc.device.check(xbc.device.lib.cc_state_space_scan_cols(xbc.device.handle, _v(xbc), _v(dt_src), int(dt_col0), _v(dt_bias), _v(a_log), _v(d_skip), _v(state), n_heads,
+                                                             n_groups, n_state, head_dim, C.byref(h)))
+    return _new(xbc.device, h, [xbc.shape()[0], n_heads * head_dim])
+
+
+def head_project_gated(x, w, n_heads, gate_src, gate_col0=0):
+    h = C.c_void_p()
+    x.device.check(x.device.lib.cc_head_project_gated(x.device.handle, _v(x), _v(w), int(n_heads), _v(gate_src), int(gate_col0), C.byref(h)))
+    return _new(x.device, h, [x.shape()[0], w.shape()[0]])
+
+
+def latent_query_append(q_src, q_col0, uk_t, n_heads, rest, freq, mag, pos0, kv_src=None, kv_col0=0, ring=None, norm_w=None, eps=0.0):
+    """the folded queries; with kv_src also writes the tokens' cache rows"""
+    h = C.c_void_p()
+    q_src.device.check(q_src.device.lib.cc_latent_query_append(q_src.device.handle, _v(q_src), int(q_col0), _v(uk_t), int(n_heads), int(rest), _v(freq), float(mag), int(pos0),
+                                                               _v(kv_src), int(kv_col0), _v(ring), _v(norm_w), float(eps), C.byref(h)))
+    return _new(q_src.device, h, [q_src.shape()[0], uk_t.shape()[0] + n_heads * rest])
+
+
+def moe_route_shared(x, router_w, correction, top, shared_gate=None, n_shared=0, n_groups=1, keep_groups=1, score=capi.ROUTE_SOFTMAX, group_top=1, renormalise=False,
+                     renorm_eps=0.0, scale=1.0):
+    """-> (ids I32 [T, top + n_shared], weights F32 [T, top + n_shared]); the last n_shared slots are the shared expert's pieces"""
+    hi, hw = C.c_void_p(), C.c_void_p()
+    rp = capi.cc_route_params(int(score), int(top), int(n_groups), int(keep_groups), int(group_top), int(renormalise), float(renorm_eps), float(scale))
+    x.device.check(x.device.lib.cc_moe_route_shared(x.device.handle, _v(x), _v(router_w), _v(correction), _v(shared_gate), int(n_shared), C.byref(rp), C.byref(hi), C.byref(hw)))
+    T = x.shape()[0]
+    return _new(x.device, hi, [T, top + n_shared]), _new(x.device, hw, [T, top + n_shared])
+
+
+def moe_experts_act(x, ids, weights, w_up, w_down, n_experts, ff, act):
+    """experts of plain units: W_down act(W_up x)"""
+    h = C.c_void_p()
+    x.device.check(x.device.lib.cc_moe_experts_act(x.device.handle, _v(x), _v(ids), _v(weights), _v(w_up), _v(w_down), int(n_experts), int(ff), int(act), C.byref(h)))
+    return _new(x.device, h, list(x.shape()))
+
+
+def feed_forward_act(x, w_up, w_down, act):
+    h = C.c_void_p()
+    x.device.check(x.device.lib.cc_feed_forward_act(x.device.handle, _v(x), _v(w_up), _v(w_down), int(act), C.byref(h)))
+    return _new(x.device, h, list(x.shape()))

@@ -28,7 +28,7 @@ import numpy as np
 from . import capi, rotary
 from .capi import CudaError, TensorError
 from .safetensors import bf16_to_f32, f32_to_bf16, read_safetensors
-from .seqmodel import SeqModel, Uploader, handle_of
+from .seqmodel import STATE_SPACE_FIELDS, SeqModel, Uploader, handle_of, parse_state_space, state_space_tensors
 from .tensor import CudaTensorDevice
 
 ARCHITECTURE = "Vuzinex"
@@ -82,10 +82,7 @@ def parse_config(conf: dict) -> dict:
                 raise TensorError(f"{at}: the right mixer has neither gate_cap nor tau")
             mixer = {"left": left, "right": right, "left_scale": float(m.get("left_scale", 1.0)), "right_scale": float(m.get("right_scale", 1.0))}
         elif L["type"] == "mamba2":
-            mixer = {k: int(m[k]) for k in ("heads", "vdim", "state", "conv")}
-            mixer["groups"], mixer["norm_groups"] = int(m.get("groups", 1)), int(m.get("norm_groups", 1))
-            if mixer["heads"] % mixer["groups"] or (mixer["heads"] * mixer["vdim"]) % mixer["norm_groups"]:
-                raise TensorError(f"{at}: groups / norm_groups do not divide the heads / the inner width")
+            mixer = parse_state_space(m, at)
         else:
             raise TensorError(f"{at}: unknown mixer type {L['type']!r}")
         mlp = L.get("mlp")
@@ -133,10 +130,7 @@ def expected_tensors(conf: dict, extras=None) -> dict:
             else:
                 t[r + "norm"] = [b["vdim"]]
         else:
-            inner, bc = m["heads"] * m["vdim"], 2 * m["groups"] * m["state"]
-            q = p + "mix."
-            t.update({q + "in": [2 * inner + bc + m["heads"], D], q + "conv": [inner + bc, m["conv"]], q + "conv.b": [inner + bc], q + "dt_bias": [m["heads"]],
-                      q + "A_log": [m["heads"]], q + "D": [m["heads"]], q + "norm": [inner], q + "o": [D, inner]})
+            t.update(state_space_tensors(m, p + "mix.", D))
         if L["mlp"]:
             ff = L["mlp"]["ff"]
             t.update({p + "norm2": [D], p + "norm2b": [D], p + "mlp.gate": [ff, D], p + "mlp.gate.b": [ff], p + "mlp.up": [ff, D], p + "mlp.up.b": [ff],
@@ -256,11 +250,10 @@ class VuzinexModel(SeqModel):
                     t["rot_freq"], lc.rot_mag = up.table(freq), mag
                 t["left_o"], t["right_o"], t["right_norm"] = up.mat(q + "o"), up.mat(r + "o"), up.vec(r + "norm")
             else:
-                q = p + "mix."
                 lc.mixer = 1
-                lc.s_heads, lc.s_vdim, lc.s_state, lc.s_groups, lc.s_conv, lc.s_norm_groups = m["heads"], m["vdim"], m["state"], m["groups"], m["conv"], m["norm_groups"]
-                t.update({"in": up.mat(q + "in"), "conv": up.mat32(q + "conv"), "conv_bias": up.vec(q + "conv.b"), "dt_bias": up.vec(q + "dt_bias"),
-                          "a_log": up.vec(q + "A_log"), "d_skip": up.vec(q + "D"), "s_norm": up.vec(q + "norm"), "s_o": up.mat(q + "o")})
+                for key, field in STATE_SPACE_FIELDS.items():
+                    setattr(lc, field, m[key])
+                t.update(up.state_space(p + "mix."))
             if mlp:
                 lc.ff = mlp["ff"]
                 t.update({"norm_c": one_plus(p + "norm2"), "norm_d": one_plus(p + "norm2b"), "gate_up": up.stack([p + "mlp.gate", p + "mlp.up"]),

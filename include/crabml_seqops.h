@@ -21,8 +21,9 @@
 extern "C" {
 #endif
 
-/* CC_ACT_SWISH: z * sigmoid(alpha * z) with alpha given beside it (cc_glu_params); the others take no constant */
-enum cc_activation { CC_ACT_NONE = 0, CC_ACT_SILU = 1, CC_ACT_GELU_TANH = 2, CC_ACT_SWISH = 3, CC_ACT_SIGMOID = 4 };
+/* CC_ACT_SWISH: z * sigmoid(alpha * z) with alpha given beside it (cc_glu_params; 1 elsewhere); the others take no constant.
+ * CC_ACT_RELU_SQUARED: max(z, 0)^2. */
+enum cc_activation { CC_ACT_NONE = 0, CC_ACT_SILU = 1, CC_ACT_GELU_TANH = 2, CC_ACT_SWISH = 3, CC_ACT_SIGMOID = 4, CC_ACT_RELU_SQUARED = 5 };
 
 /* x (any shape) = 0 */
 CC_API int cc_tensor_zero(cc_device* dev, const cc_view* x);
@@ -46,7 +47,8 @@ CC_API int cc_group_rms_norm(cc_device* dev, const cc_view* dst, const cc_view* 
  * mean.  dst, x: [rows, cols]; w, b: [cols] (b NULL: no bias).  dst may be x. */
 CC_API int cc_layer_norm(cc_device* dev, const cc_view* dst, const cc_view* x, const cc_view* w, const cc_view* b, float eps);
 /* dst = x * act(gate) with every one of `groups` equal consecutive parts of the row then divided by its own root mean square, times w[:]:
- * the gate comes BEFORE the norm (cc_gated_head_rms_norm gates after it).  All [rows, cols]; w: [cols].  dst may be x. */
+ * the gate comes BEFORE the norm (cc_gated_head_rms_norm gates after it).  All [rows, cols]; w: [cols].  dst may be x.  gate may be the first
+ * columns of the rows of a wider matrix (row stride > cols). */
 CC_API int cc_gated_group_rms_norm(cc_device* dev, const cc_view* dst, const cc_view* x, const cc_view* gate, const cc_view* w, int32_t groups, float eps,
                                    int32_t gate_act);
 /* PolyNorm, in place on z [rows, cols]: z <- a N(z) + b N(z^2) + c N(z^3) + e with coef = {a, b, c, e}; powers are taken element by
@@ -62,6 +64,10 @@ CC_API int cc_gated_sum(cc_device* dev, const cc_view* dst, int32_t accumulate, 
 CC_API int cc_split_cols(cc_device* dev, const cc_view* src, int32_t n_parts, const int32_t* widths, cc_buf** outs);
 /* gate = act(gate) * up, elementwise (the inner step of a gated feed-forward, exact 32-bit activation) */
 CC_API int cc_glu_inplace(cc_device* dev, const cc_view* gate, const cc_view* up, int32_t act);
+/* x = act(x), elementwise */
+CC_API int cc_activate_inplace(cc_device* dev, const cc_view* x, int32_t act);
+/* x = cap * tanh(x / cap), elementwise (capped logits); cap > 0 */
+CC_API int cc_softcap_inplace(cc_device* dev, const cc_view* x, float cap);
 /* The same step on ONE product of the stacked matrix [W_gate ; W_up]: src [rows, 2 * ff] holds gate | up side by side;
  * out[r, c] = act(src[r, c] + bias[c]) * (src[r, ff + c] + bias[ff + c]) ; bias: [2 * ff] or NULL.  out: [rows, ff]. */
 CC_API int cc_glu_halves(cc_device* dev, const cc_view* src, const cc_view* bias, int32_t act, cc_buf** out);
@@ -99,6 +105,10 @@ CC_API int cc_short_conv_biases(cc_device* dev, const cc_view* x, const cc_view*
                                 cc_buf** out);
 /* cc_short_conv with a bias per channel added to the sum before the activation (bias: [C] or NULL) */
 CC_API int cc_short_conv_bias(cc_device* dev, const cc_view* x, const cc_view* w, const cc_view* bias, const cc_view* tail, int32_t act, cc_buf** out);
+
+/* cc_short_conv_bias on the columns col0 .. col0 + C of a wider matrix src [T, >= col0 + C] (w: [C, K]): a block of one stacked product's
+ * result, read where it lies */
+CC_API int cc_short_conv_cols(cc_device* dev, const cc_view* src, int32_t col0, const cc_view* w, const cc_view* bias, const cc_view* tail, int32_t act, cc_buf** out);
 
 /* ---- gated delta rule ------------------------------------------------------------------------------------------------------ */
 /* One sequence, T new tokens.  q, k: [T, n_kv * dk] (already normalised), v: [T, n_heads * dv]; a, b: [T, n_heads] raw projections;
@@ -165,6 +175,9 @@ CC_API int cc_decayed_linear_attention(cc_device* dev, const cc_view* q, const c
  * out: [T, H * P]. */
 CC_API int cc_state_space_scan(cc_device* dev, const cc_view* xbc, const cc_view* dt, const cc_view* dt_bias, const cc_view* a_log, const cc_view* d_skip,
                                const cc_view* state, int32_t n_heads, int32_t n_groups, int32_t n_state, int32_t head_dim, cc_buf** out);
+/* cc_state_space_scan with the raw step sizes in the columns dt_col0 .. dt_col0 + H of a wider matrix dt_src [T, >= dt_col0 + H] */
+CC_API int cc_state_space_scan_cols(cc_device* dev, const cc_view* xbc, const cc_view* dt_src, int32_t dt_col0, const cc_view* dt_bias, const cc_view* a_log,
+                                    const cc_view* d_skip, const cc_view* state, int32_t n_heads, int32_t n_groups, int32_t n_state, int32_t head_dim, cc_buf** out);
 /* Retention: linear attention with one fixed decay per head, no softmax and no denominator.  q, k: [T, H * dk], v: [T, H * dv];
  * decay: [H]; state: [H, dk, dv].
  *   S = decay[h] S + (k_scale k) v^T ; out = S^T q */
@@ -226,6 +239,16 @@ CC_API int cc_latent_ring_append(cc_device* dev, const cc_view* ring, const cc_v
 CC_API int cc_head_project(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, int32_t rest, const cc_view* freq, float mag, int64_t pos0,
                            cc_buf** out);
 
+/* cc_head_project without carried columns and with a gate on the result: out[t, h] = (W_h x[t, h]) * sigmoid(g[t, h]), g the columns
+ * gate_col0 .. gate_col0 + heads * n_out of gate_src's rows (a block of a stacked product's result) */
+CC_API int cc_head_project_gated(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, cc_buf** out);
+/* What a decoding pass of latent attention does between its projections and the scores, in one kernel: the queries' fold
+ * (cc_head_project with carried columns rotated on the way; queries in the columns q_col0 .. of q_src's rows, uk_t: [heads * rank, dim])
+ * and the cache rows of the same tokens (cc_latent_ring_append; raw rows in the columns kv_col0 .. of kv_src).  kv_src NULL: nothing is
+ * appended (a layer that reads another layer's cache; ring and norm_w are ignored).  out: [T, heads * (rank + rest)]. */
+CC_API int cc_latent_query_append(cc_device* dev, const cc_view* q_src, int32_t q_col0, const cc_view* uk_t, int32_t n_heads, int32_t rest, const cc_view* freq, float mag,
+                                  int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps, cc_buf** out);
+
 /* out[j, h] = [ a[j, h] | shared[j, col0 : col0 + rest] ]: a: [rows, heads * dim]; shared: [>= rows, cols] (its first `rows` rows are used);
  * out: [rows, heads * (dim + rest)].  Builds per-head keys out of their own part and a part all heads share (a latent cache's rotated columns). */
 CC_API int cc_head_concat_shared(cc_device* dev, const cc_view* a, const cc_view* shared, int32_t n_heads, int32_t col0, int32_t rest, cc_buf** out);
@@ -246,9 +269,15 @@ typedef struct cc_route_params {
     int32_t group_top;           /* a group's score is the sum of its group_top largest choice scores (1: its largest) */
     int32_t renormalise;         /* != 0: the chosen weights are divided by (their sum + renorm_eps) */
     float renorm_eps;
+    float scale;                 /* factor on the chosen weights, after the renormalisation; 0 counts as 1 */
 } cc_route_params;
 CC_API int cc_moe_route_ex(cc_device* dev, const cc_view* x, const cc_view* router_w, const cc_view* correction, const cc_route_params* params,
                            cc_buf** ids_out, cc_buf** weights_out);
+/* cc_moe_route_ex with n_shared more slots per token behind the chosen ones: ids E, E + 1, ... (E experts), all with the weight
+ * sigmoid(shared_gate . x) (shared_gate: [D], or NULL: weight 1).  They stand for a shared expert that every token uses, cut into pieces of the
+ * experts' hidden width and stacked behind them.  ids_out, weights_out: [T, top + n_shared]. */
+CC_API int cc_moe_route_shared(cc_device* dev, const cc_view* x, const cc_view* router_w, const cc_view* correction, const cc_view* shared_gate, int32_t n_shared,
+                               const cc_route_params* params, cc_buf** ids_out, cc_buf** weights_out);
 /* the gated unit of an expert: act(min(g, limit)) * (clamp(u, -limit, limit) + up_shift); limit <= 0: nothing is clamped */
 typedef struct cc_glu_params {
     int32_t act;                 /* cc_activation */
@@ -262,6 +291,11 @@ CC_API int cc_moe_experts_glu(cc_device* dev, const cc_view* x, const cc_view* i
  * w_gate, w_up: [E * ff, D]; w_down: [E * D, ff] (expert-major stacks; F32 or BF16).  out: [T, D]. */
 CC_API int cc_moe_experts(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_gate, const cc_view* w_up,
                           const cc_view* w_down, int32_t n_experts, int32_t ff, int32_t act, cc_buf** out);
+/* experts of plain units: out[t] = sum_s weights[t, s] * W_down[ids[t, s]] act(W_up[ids[t, s]] x[t]) */
+CC_API int cc_moe_experts_act(cc_device* dev, const cc_view* x, const cc_view* ids, const cc_view* weights, const cc_view* w_up, const cc_view* w_down, int32_t n_experts,
+                              int32_t ff, int32_t act, cc_buf** out);
+/* the same unit for every token: out = W_down act(W_up x) ; w_up: [ff, D], w_down: [D, ff], both F32 or both BF16 */
+CC_API int cc_feed_forward_act(cc_device* dev, const cc_view* x, const cc_view* w_up, const cc_view* w_down, int32_t act, cc_buf** out);
 
 #ifdef __cplusplus
 }
