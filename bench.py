@@ -49,6 +49,10 @@ WORKLOADS = {
     "lifesun-w1024": ("LIFESUN", "BF16", "BF16"),
     "lifesun-w2048": ("LIFESUN", "BF16", "BF16"),
     "lifesun-w4096": ("LIFESUN", "BF16", "BF16"),
+    # the Papunex family at the same layer sizes, beside the Meresun and Vuzinex stacks of equal width and depth; see run_papunex
+    "papunex-w1024": ("PAPUNEX", "BF16", "BF16"),
+    "papunex-w2048": ("PAPUNEX", "BF16", "BF16"),
+    "papunex-w4096": ("PAPUNEX", "BF16", "BF16"),
 }
 # dram bytes per megakernel launch from the committed ncu --set full capture (profiles/); None until captured
 TRAFFIC = {("llama2-7b-q8_0", 1): 7040893000 + 49879296}     # profiles/r02p_mega_ring_q8_0_ncu_raw.csv (mega_ring_kernel: dram__bytes_read.sum + dram__bytes_write.sum)
@@ -823,6 +827,110 @@ def run_lifesun(args, rank, world, local_rank):
     print(json.dumps(line))
 
 
+def papunex_bench_config(width: int, vocab: int = 32000):
+    """four layers whose active feed-forward width is 3 x width per token, as in the Meresun and Vuzinex stacks: latent attention (128 + 64 wide
+    query heads over a latent of 512, causal) with a dense feed-forward, two state-space layers (heads of 64, 128 states, 4 taps) and latent
+    attention over the first layer's cache, each of the three with 16 experts of width/2 (top 4) and a shared expert of the model's width"""
+    att = {"heads": width // 128, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": {"dims": 64, "base": 10000.0}}
+    ssm = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    dense = {"kind": "dense", "ff": 3 * width}
+    moe = {"kind": "moe", "expert": {"ff": width // 2}, "router": {"experts": 16, "top": 4, "scale": 2.5}, "shared": {"ff": width}}
+    layers = [{"type": "latent_attention", "mixer": att, "mlp": dense}, {"type": "mamba2", "mixer": ssm, "mlp": moe}, {"type": "mamba2", "mixer": ssm, "mlp": moe},
+              {"type": "latent_attention", "mixer": dict(att, kv_from=0), "mlp": moe}]
+    return {"architecture": "Papunex", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": layers}
+
+
+def time_papunex_kernels(dev, width, T):
+    """The feed-forward steps of the Papunex family alone at the bench's sizes, beside the like steps of the Meresun stack (gated experts of equal
+    width), for a prompt of T rows (floating-point operations per second) and for one decoded row (weight bytes per second)."""
+    from crabml_b200 import CudaTensor, capi, seqops
+    from crabml_b200.safetensors import f32_to_bf16
+    rng = np.random.default_rng(SEED)
+
+    def rand(*shape):
+        return CudaTensor.new(rng.standard_normal(shape).astype(np.float32), list(shape), dev)
+
+    def mat(*shape):
+        a = (rng.standard_normal(shape) / np.sqrt(shape[-1])).astype(np.float32)
+        return CudaTensor.from_cpu(np.ascontiguousarray(f32_to_bf16(a).reshape(shape)), list(shape), capi.BF16, dev)
+    out = {}
+    flush = rand(48 * 1024 * 1024)                                     # 192 MB: read and written between timed calls, so that no call finds its weights in L2
+
+    def timed(name, f, reps=5, **what):
+        f()
+        ms = 0.0
+        for _ in range(reps):
+            seqops.activate_inplace(flush, capi.ACT_NONE)
+            dev.synchronize(); dev.timer_begin()
+            f()
+            ms += dev.timer_end()
+        out[name] = dict(what, ms=ms / reps)
+        if "flop" in what:
+            out[name]["flop_per_s"] = what["flop"] / (ms / reps * 1e-3)
+        if "bytes" in what:
+            out[name]["bytes_per_s"] = what["bytes"] / (ms / reps * 1e-3)
+    D, E, ff, top, ns = width, 16, width // 2, 4, 2
+    n_all = E + ns
+    wg, wu, wd = mat(n_all * ff, D), mat(n_all * ff, D), mat(n_all * D, ff)
+    router, sg = rand(E, D), rand(D)
+    up3, down3 = mat(3 * D, D), mat(D, 3 * D)
+    for rows, tag in ((T, "prompt"), (1, "decode")):
+        x = rand(rows, D)
+        slots = top + ns
+        ids, wts = seqops.moe_route_shared(x, router, None, top, shared_gate=sg, n_shared=ns, renormalise=True, renorm_eps=1e-20, scale=2.5)
+        plain, gated = {"rows": rows, "slots": slots, "ff": ff}, {"rows": rows, "slots": slots, "ff": ff}
+        if rows > 1:
+            plain["flop"], gated["flop"] = 2 * rows * slots * 2 * D * ff, 2 * rows * slots * 3 * D * ff
+        else:
+            plain["bytes"], gated["bytes"] = slots * 2 * D * ff * 2, slots * 3 * D * ff * 2
+        timed(f"{tag}: experts of plain units + shared pieces", lambda: seqops.moe_experts_act(x, ids, wts, wu, wd, n_all, ff, capi.ACT_RELU_SQUARED), **plain)
+        timed(f"{tag}: gated experts (closest model)", lambda: seqops.moe_experts_glu(x, ids, wts, wg, wu, wd, n_all, ff, capi.ACT_SILU), **gated)
+        timed(f"{tag}: router with shared gate", lambda: seqops.moe_route_shared(x, router, None, top, shared_gate=sg, n_shared=ns, renormalise=True, renorm_eps=1e-20, scale=2.5), rows=rows)
+        timed(f"{tag}: router (closest model)", lambda: seqops.moe_route_ex(x, router, None, top, renormalise=True), rows=rows)
+        dense = {"rows": rows, "ff": 3 * D}
+        dense.update({"flop": 2 * rows * 2 * D * 3 * D} if rows > 1 else {"bytes": 2 * D * 3 * D * 2})
+        timed(f"{tag}: dense feed-forward of plain units", lambda: seqops.feed_forward_act(x, up3, down3, capi.ACT_RELU_SQUARED), **dense)
+        timed(f"{tag}: two dense products of the same sizes", lambda: down3.matmul_vec(up3.matmul_vec(x)), **dense)
+    return out
+
+
+def run_papunex(args, rank, world, local_rank):
+    """Prefill and decode throughput of the Papunex family at real layer sizes, beside the closest existing models -- the Meresun stack (latent
+    attention, routed feed-forward) and the Vuzinex stack (state-space layers) of the same width, depth and active feed-forward width -- through
+    the same step function and slots; then the family's feed-forward steps alone beside the like steps of the closest model."""
+    from crabml_b200 import CudaTensorDevice, meresun, papunex, vuzinex
+    if rank != 0:
+        return
+    width = int(args.workload.split("-w")[1])
+    Tp, K, W = args.prefill_tokens, args.steps, args.warmup
+    rng = np.random.default_rng(SEED)
+    prompt = [int(v) for v in rng.integers(0, 32000, Tp)]
+    sampler = ClockSampler(local_rank); sampler.start()
+    out = {}
+    for name, mod, cls, raw in (("papunex", papunex, "PapunexModel", papunex_bench_config(width)), ("meresun", meresun, "MeresunModel", meresun_bench_config(width)),
+                                ("vuzinex", vuzinex, "VuzinexModel", vuzinex_bench_config(width))):
+        conf = mod.parse_config(raw)
+        dev = CudaTensorDevice(local_rank, lazy=0)
+        weights = mod.random_weights(conf, SEED)
+        model = getattr(mod, cls)(dev, conf, weights, "bfloat16", chunk=args.zatorax_chunk, max_seq=Tp + K + W + 8)
+        params = sum(int(np.prod(np.shape(a))) for a in weights.values())
+        del weights
+        out[name] = measure_seq_model(dev, model, prompt, K, W, params)
+        model.close()
+        if name == "papunex":
+            out["feed_forward_steps"] = time_papunex_kernels(dev, width, min(Tp, 2048))
+        dev.close()
+    clocks = sampler.stop()
+    z = out["papunex"]
+    line = {"metric": "decode_tokens_per_s", "value": z["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": z["decode_ms_per_token"],
+            "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 matrices and product inputs, f32 everything else", "data": "synthetic",
+            "config": {"workload": args.workload, "model": papunex_bench_config(width), "prefill_tokens": Tp, "chunk": args.zatorax_chunk,
+                       "closest_models": {"meresun": meresun_bench_config(width), "vuzinex": vuzinex_bench_config(width)}},
+            "e2e": {"value": 1e3 / z["decode_wall_ms_per_token"], "unit": "tok/s", "h2d_bytes_per_step": 8, "d2h_bytes_per_step": 32000 * 4},
+            "gpu_launches": int(z["decode_launches_per_token"] * K), "detail": out, "clocks": clocks}
+    print(json.dumps(line))
+
+
 def run_zatorax(args, rank, world, local_rank):
     """Prefill and decode throughput of the Zatorax family at real layer sizes, beside the closest existing model -- a llama stack of the
     same width, depth, head layout and ACTIVE feed-forward width (Q8_0 weights, its serving format) -- through each family's runner.
@@ -900,7 +1008,7 @@ def main():
     ap.add_argument("--no-also", action="store_true", help="skip the second (Q4_0) measurement of the default run")
     ap.add_argument("--multi", default="sharded", choices=["sharded", "replicas"], help="N > 1: shard one token stream (strong scaling, default) or run N independent replicas")
     ap.add_argument("--comm", default="p2p", choices=["p2p", "nccl"], help="exchange transport of the sharded path: one-shot NVLink peer stores (default) or the NCCL baseline")
-    ap.add_argument("--zatorax-chunk", type=int, default=512, help="zatorax / meresun / vuzinex / lifesun workloads: longest run of prompt tokens one pass takes")
+    ap.add_argument("--zatorax-chunk", type=int, default=512, help="zatorax / meresun / vuzinex / lifesun / papunex workloads: longest run of prompt tokens one pass takes")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -915,6 +1023,8 @@ def main():
         run_vuzinex(args, rank, world, local_rank)
     elif args.workload.startswith("lifesun-"):
         run_lifesun(args, rank, world, local_rank)
+    elif args.workload.startswith("papunex-"):
+        run_papunex(args, rank, world, local_rank)
     elif args.workload.endswith("-prefill"):
         run_prefill(args, rank, world, local_rank)
     else:

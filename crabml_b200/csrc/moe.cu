@@ -38,28 +38,63 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
         if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
     }
 }
-#define RT_WARPS 8
-// one CTA per token: its warps share the experts' logits (a warp per expert, lanes striding D), then warp 0 does the softmax and the choice
-__global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const float* __restrict__ x, const float* __restrict__ wr, const float* __restrict__ corr,
-                                                                  int* __restrict__ ids, float* __restrict__ wts, int T, int D, int E, int top, int n_groups, int keep,
-                                                                  int renorm, int score_fn, int group_top, float renorm_eps, float scale, const float* __restrict__ wsg, int n_shared) {
+#define RT_WARPS 16
+struct RouteArgs {
+    const float *x, *wr, *corr, *wsg;      // corr: NULL or [E]; wsg: NULL or the shared gate's row [D]
+    int* ids;
+    float* wts;
+    int T, D, E, top, n_groups, keep, renorm, score_fn, group_top, n_shared, vec;
+    float renorm_eps, scale;
+};
+// one CTA per TOK tokens: its warps share the experts' logits (a warp per expert and all TOK tokens: lanes striding D in 16-byte pieces, or element
+// by element when D or the pointers do not allow them; then the butterfly), then warp tt does token tt's softmax and choice.  The order of a
+// logit's sum does not depend on TOK.
+template <int TOK>
+__global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(RouteArgs a) {
     extern __shared__ float rt_sm[];
+    __shared__ float sg_sm[TOK];                           // the shared gate's logit: row E of the same products
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x;
-    float* s = rt_sm;
-    float* c = s + E;
-    float* gs = c + E;
-    const float* xr = x + (int64_t)t * D;
-    __shared__ float sg;                                   // the shared gate's logit: row E of the same products
+    const int t0 = blockIdx.x * TOK, D = a.D, E = a.E, top = a.top, n_groups = a.n_groups, keep = a.keep, group_top = a.group_top, score_fn = a.score_fn, n_shared = a.n_shared;
+    const float *corr = a.corr, *wsg = a.wsg;
+    int* ids = a.ids;
+    float* wts = a.wts;
+    const int per_token = 2 * E + (n_groups > 1 ? n_groups : 0);
     for (int e = warp; e < E + (wsg ? 1 : 0); e += RT_WARPS) {
-        const float* w = e < E ? wr + (int64_t)e * D : wsg;
-        float acc = 0.0f;
-        for (int d = lane; d < D; d += 32) acc = fmaf(w[d], xr[d], acc);
-        acc = warp_sum(acc);
-        if (lane == 0) *(e < E ? s + e : &sg) = acc;
+        const float* w = e < E ? a.wr + (int64_t)e * D : wsg;
+        const float* xr[TOK];
+        float acc[TOK];
+#pragma unroll
+        for (int tt = 0; tt < TOK; tt++) { xr[tt] = a.x + (int64_t)min(t0 + tt, a.T - 1) * D; acc[tt] = 0.0f; }
+        if (a.vec) {
+#pragma unroll 4
+            for (int d = lane * 4; d < D; d += 128) {
+                const float4 wv = *(const float4*)(w + d);
+#pragma unroll
+                for (int tt = 0; tt < TOK; tt++) {
+                    const float4 xv = *(const float4*)(xr[tt] + d);
+                    acc[tt] = fmaf(wv.x, xv.x, acc[tt]); acc[tt] = fmaf(wv.y, xv.y, acc[tt]); acc[tt] = fmaf(wv.z, xv.z, acc[tt]); acc[tt] = fmaf(wv.w, xv.w, acc[tt]);
+                }
+            }
+        } else {
+            for (int d = lane; d < D; d += 32) {
+                const float wv = w[d];
+#pragma unroll
+                for (int tt = 0; tt < TOK; tt++) acc[tt] = fmaf(wv, xr[tt][d], acc[tt]);
+            }
+        }
+#pragma unroll
+        for (int tt = 0; tt < TOK; tt++) {
+            const float v = warp_sum(acc[tt]);
+            if (lane == 0) *(e < E ? rt_sm + tt * per_token + e : sg_sm + tt) = v;
+        }
     }
     __syncthreads();
-    if (warp != 0) return;
+    const int t = t0 + warp;
+    if (warp >= TOK || t >= a.T) return;
+    float* s = rt_sm + warp * per_token;
+    float* c = s + E;
+    float* gs = c + E;
+    const float sg = sg_sm[warp];
     if (score_fn == CC_ROUTE_SIGMOID) {
         for (int e = lane; e < E; e += 32) { const float v = 1.0f / (1.0f + expf(-s[e])); s[e] = v; c[e] = corr ? v + corr[e] : v; }
     } else {
@@ -119,8 +154,8 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const float* _
         __syncwarp();
     }
     if (lane == 0) {
-        if (renorm) for (int r = 0; r < top; r++) wts[(int64_t)t * slots + r] /= wsum + renorm_eps;
-        if (scale != 1.0f) for (int r = 0; r < top; r++) wts[(int64_t)t * slots + r] *= scale;
+        if (a.renorm) for (int r = 0; r < top; r++) wts[(int64_t)t * slots + r] /= wsum + a.renorm_eps;
+        if (a.scale != 1.0f) for (int r = 0; r < top; r++) wts[(int64_t)t * slots + r] *= a.scale;
     }
     for (int r = lane; r < n_shared; r += 32) {
         ids[(int64_t)t * slots + top + r] = E + r;
@@ -153,14 +188,17 @@ extern "C" CC_API int cc_moe_route_shared(cc_device* dev, const cc_view* x, cons
     if (rc) { cc_tensor_release(ids); return rc; }
     *ids_out = ids; *weights_out = wts;
     if (T == 0) return CC_OK;
-    const size_t smem = (size_t)(2 * E + (n_groups > 1 ? n_groups : 0)) * 4;
-    if (smem > 200 * 1024) return cc_fail(dev, CC_ERR_UNSUPPORTED, "moe_route: %lld experts need %zu bytes of shared memory", (long long)E, smem);
-    if (smem > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    moe_route_kernel<<<(unsigned)T, RT_WARPS * 32, smem, dev->stream>>>((const float*)x->buf->plane[0], (const float*)router_w->buf->plane[0],
-                                                                                                     correction ? (const float*)correction->buf->plane[0] : nullptr,
-                                                                                                     (int*)ids->base, (float*)wts->base, (int)T, (int)D, (int)E, top, n_groups,
-                                                                                                     keep_groups, renormalise, rp->score, group_top, rp->renorm_eps, scale,
-                                                                                                     shared_gate ? (const float*)shared_gate->buf->plane[0] : nullptr, n_shared);
+    const float* xp = (const float*)x->buf->plane[0];
+    const float* rp_w = (const float*)router_w->buf->plane[0];
+    const float* sgp = shared_gate ? (const float*)shared_gate->buf->plane[0] : nullptr;
+    const RouteArgs a = {xp, rp_w, correction ? (const float*)correction->buf->plane[0] : nullptr, sgp, (int*)ids->base, (float*)wts->base, (int)T, (int)D, (int)E, top, n_groups, keep_groups,
+                         renormalise, rp->score, group_top, n_shared, D % 4 == 0 && (((uintptr_t)xp | (uintptr_t)rp_w | (uintptr_t)sgp) & 15) == 0 ? 1 : 0, rp->renorm_eps, scale};
+    const size_t one = (size_t)(2 * E + (n_groups > 1 ? n_groups : 0)) * 4;
+    if (one > 200 * 1024) return cc_fail(dev, CC_ERR_UNSUPPORTED, "moe_route: %lld experts need %zu bytes of shared memory", (long long)E, one);
+    const bool tiled = T >= 128 && 4 * one <= 48 * 1024;              // a pass of many rows: every router row is read once for four tokens
+    if (!tiled && one > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_route_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)one));
+    if (tiled) moe_route_kernel<4><<<(unsigned)((T + 3) / 4), RT_WARPS * 32, 4 * one, dev->stream>>>(a);
+    else moe_route_kernel<1><<<(unsigned)T, RT_WARPS * 32, one, dev->stream>>>(a);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
@@ -242,12 +280,14 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const float* __restrict__
     __syncthreads();
     const int d = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (d >= D) return;
-    float acc = 0.0f;
+    float acc = 0.0f;                     // a lane's weighted share of all slots, in slot order; the butterfly comes last
+#pragma unroll 4
     for (int s = 0; s < top; s++) {
         const int e = ids ? moe_clamp(ids[(int64_t)t * top + s], E) : 0;
-        const float p = warp_sum(moe_dot<WT, VEC>(wd + ((int64_t)e * D + d) * ff, md_sm + s * ff, ff, lane));
+        const float p = moe_dot<WT, VEC>(wd + ((int64_t)e * D + d) * ff, md_sm + s * ff, ff, lane);
         acc = wts ? fmaf(wts[(int64_t)t * top + s], p, acc) : acc + p;
     }
+    acc = warp_sum(acc);
     if (lane == 0) out[(int64_t)t * D + d] = acc;
 }
 
