@@ -38,7 +38,6 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
         if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
     }
 }
-#define RT_WARPS 16
 struct RouteArgs {
     const float *x, *wr, *corr, *wsg;      // corr: NULL or [E]; wsg: NULL or the shared gate's row [D]
     int* ids;
@@ -50,16 +49,16 @@ struct RouteArgs {
 // by element when D or the pointers do not allow them; then the butterfly), then warp tt does token tt's softmax and choice.  The order of a
 // logit's sum does not depend on TOK.
 template <int TOK>
-__global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(RouteArgs a) {
+__global__ void __launch_bounds__(TOK == 1 ? 1024 : 512) moe_route_kernel(RouteArgs a) {
     extern __shared__ float rt_sm[];
     __shared__ float sg_sm[TOK];                           // the shared gate's logit: row E of the same products
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
     const int t0 = blockIdx.x * TOK, D = a.D, E = a.E, top = a.top, n_groups = a.n_groups, keep = a.keep, group_top = a.group_top, score_fn = a.score_fn, n_shared = a.n_shared;
     const float *corr = a.corr, *wsg = a.wsg;
     int* ids = a.ids;
     float* wts = a.wts;
     const int per_token = 2 * E + (n_groups > 1 ? n_groups : 0);
-    for (int e = warp; e < E + (wsg ? 1 : 0); e += RT_WARPS) {
+    for (int e = warp; e < E + (wsg ? 1 : 0); e += n_warps) {
         const float* w = e < E ? a.wr + (int64_t)e * D : wsg;
         const float* xr[TOK];
         float acc[TOK];
@@ -197,8 +196,12 @@ extern "C" CC_API int cc_moe_route_shared(cc_device* dev, const cc_view* x, cons
     if (one > 200 * 1024) return cc_fail(dev, CC_ERR_UNSUPPORTED, "moe_route: %lld experts need %zu bytes of shared memory", (long long)E, one);
     const bool tiled = T >= 128 && 4 * one <= 48 * 1024;              // a pass of many rows: every router row is read once for four tokens
     if (!tiled && one > 48 * 1024) CC_CUDA(dev, cudaFuncSetAttribute(moe_route_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)one));
-    if (tiled) moe_route_kernel<4><<<(unsigned)((T + 3) / 4), RT_WARPS * 32, 4 * one, dev->stream>>>(a);
-    else moe_route_kernel<1><<<(unsigned)T, RT_WARPS * 32, one, dev->stream>>>(a);
+    // as many warps as share the rows evenly in the fewest rounds (at most 16 per CTA of four tokens, 32 per CTA of one)
+    const int64_t rows = E + (shared_gate ? 1 : 0), most = tiled ? 16 : 32, rounds = (rows + most - 1) / most;
+    const int64_t even = (rows + rounds - 1) / rounds;
+    const unsigned threads = 32 * (unsigned)(even < 4 ? 4 : even);
+    if (tiled) moe_route_kernel<4><<<(unsigned)((T + 3) / 4), threads, 4 * one, dev->stream>>>(a);
+    else moe_route_kernel<1><<<(unsigned)T, threads, one, dev->stream>>>(a);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
