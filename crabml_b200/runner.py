@@ -184,7 +184,7 @@ def synth_scale(dtype, k):
 
 def synthetic_weights(device: CudaTensorDevice, conf: LlamaConfig, wtype: int, classifier_type: int | None = None,
                       seed: int = 0x5EED, plan: "sharding.ShardPlan | None" = None):
-    """Valid, non-degenerate random blocks generated ON the device (never shipped through gpurun).
+    """Valid, non-degenerate random blocks generated ON the device, so that they never cross the host.
     plan: generate only this rank's shard of every tensor (same bytes as the corresponding slice of the full model)."""
     ct = wtype if classifier_type is None else classifier_type
     dim, hid, kv = conf.embedding_dim, conf.hidden_dim, conf.head_size() * conf.n_kv_heads

@@ -138,8 +138,8 @@ def test_the_cache_is_sized_by_the_token_budget(dev):
     m.close()
 
 
-def _recall_model(T, j_star):
-    """One attention layer (one head) whose scores are 0 but for the key of token 1, which every query scores with about 90; its value carries a
+def _recall_model():
+    """One attention layer (one head) whose scores are 0 but for the key of token id 1, which every query scores with about 90; its value carries a
     mark to the logits.  -> conf, weights"""
     conf = config([latent(heads=1, dim=2, rot_dim=2, vdim=2, kv_rank=2, scale=1.0, base=10.0, mlp=None)], width=4, vocab=3, eps=1e-6, embed_scale=1.0, softcap=0)
     w = {n: np.zeros(s, np.float32) for n, s in papunex.expected_tensors(papunex.parse_config(conf)).items()}
@@ -161,7 +161,7 @@ def _recall_model(T, j_star):
 @pytest.mark.parametrize("j_star", [0, 255, 256, 300])
 def test_a_far_token_decides_prompts_and_decoded_tokens(dev, dtype, j_star):
     T = 900
-    conf, w = _recall_model(T, j_star)
+    conf, w = _recall_model()
     c, w, m = build(dev, conf, 0, dtype, weights=w)
     toks = [0] * T
     toks[j_star] = 1
