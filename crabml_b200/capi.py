@@ -159,12 +159,28 @@ class cpr_layer_weights(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in CPR_WEIGHT_FIELDS]
 
 
-class cc_route_params(C.Structure):              # include/crabml_seqops.h
-    _fields_ = [(n, C.c_int32) for n in ("score", "top", "n_groups", "keep_groups", "group_top", "renormalise")] + [("renorm_eps", C.c_float), ("scale", C.c_float)]
-
-
 class cc_glu_params(C.Structure):
     _fields_ = [("act", C.c_int32), ("alpha", C.c_float), ("limit", C.c_float), ("up_shift", C.c_float)]
+
+
+class cvd_layer_config(C.Structure):            # include/crabml_vadodra.h
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "rot_dim", "kv_rank", "kv_from")] + \
+               [("scale", C.c_float), ("rot_mag", C.c_float), ("ff", C.c_int32), ("glu", cc_glu_params)]
+
+
+class cvd_config(C.Structure):
+    _fields_ = [("n_layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("norm_eps", C.c_float), ("chunk", C.c_int32), ("max_seq", C.c_int32)]
+
+
+CVD_WEIGHT_FIELDS = ("norm", "h_stack", "o_stack", "q_norm", "k_norm", "rot_freq", "dkv_norm", "uk", "uv", "uk_t", "uv_f32")
+
+
+class cvd_layer_weights(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in CVD_WEIGHT_FIELDS]
+
+
+class cc_route_params(C.Structure):              # include/crabml_seqops.h
+    _fields_ = [(n, C.c_int32) for n in ("score", "top", "n_groups", "keep_groups", "group_top", "renormalise")] + [("renorm_eps", C.c_float), ("scale", C.c_float)]
 
 
 _lib = None
@@ -310,6 +326,14 @@ def load_library(build_if_missing: bool = True):
         "cc_moe_route_shared": (i32, [vp, pv, pv, pv, pv, i32, C.POINTER(cc_route_params), pp, pp]),
         "cc_moe_experts_act": (i32, [vp, pv, pv, pv, pv, pv, i32, i32, i32, pp]),
         "cc_feed_forward_act": (i32, [vp, pv, pv, pv, i32, pp]),
+        "cc_head_gate_cols": (i32, [vp, pv, pv, i32, i32, i32]),
+        "cc_qk_prepare_append_cols": (i32, [vp, pv, i32, i32, i32, pv, pv, i32, pv, pv, f32, pv, i32, i32, f32, i64, i32, i32, i32, i32, pp]),
+        "cc_head_project_head_gated": (i32, [vp, pv, pv, i32, pv, i32, pp]),
+        "cc_latent_query_append_paired": (i32, [vp, pv, i32, pv, i32, i32, pv, i32, f32, i64, pv, i32, pv, pv, f32, pp]),
+        "cc_latent_prepare_append": (i32, [vp, pv, i32, i32, i32, i32, pv, i32, f32, i64, pv, i32, pv, pv, f32, pp]),
+        "cc_layer_norm_product": (i32, [vp, pv, pv, pv, f32, pv, pp]),
+        "cc_joined_product_accumulate": (i32, [vp, pv, pv, pv, pv, i32, i32, i32, C.POINTER(cc_glu_params)]),
+        "cvd_runner_create": (i32, [vp, C.POINTER(cvd_config), C.POINTER(cvd_layer_config), C.POINTER(cvd_layer_weights), vp, vp, vp, pp]),
         "cpr_runner_create": (i32, [vp, C.POINTER(cpr_config), C.POINTER(cpr_layer_config), C.POINTER(cpr_layer_weights), vp, vp, vp, pp]),
         "clr_runner_create": (i32, [vp, C.POINTER(clr_config), C.POINTER(clr_layer_config), C.POINTER(clr_layer_weights), vp, vp, vp, vp, vp, pp]),
         "cvr_runner_create": (i32, [vp, C.POINTER(cvr_config), C.POINTER(cvr_layer_config), C.POINTER(cvr_layer_weights), vp, vp, vp, vp, pp]),

@@ -18,3 +18,8 @@ __device__ __forceinline__ float act_apply(float z, int act, float alpha = 1.0f)
     }
     return z;
 }
+// the gated unit: act(min(g, limit)) * (clamp(u, -limit, limit) + up_shift); limit <= 0 clamps nothing
+__device__ __forceinline__ float glu_apply(float g, float u, const cc_glu_params P) {
+    if (P.limit > 0.0f) { g = fminf(g, P.limit); u = fminf(fmaxf(u, -P.limit), P.limit); }
+    return act_apply(g, P.act, P.alpha) * (u + P.up_shift);
+}

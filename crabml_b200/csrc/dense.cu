@@ -22,7 +22,7 @@ __device__ __forceinline__ float dn_load_w(const uint16_t* w, int64_t i) { retur
 
 // grid: (ceil(m / 64), ceil(b / 64)).  Thread (ty, tx) of a 16 x 16 layout owns batch rows ty*4.. and weight rows tx*4.. of the tile.
 template <class WT, bool ROUND_X>
-__global__ void __launch_bounds__(DN_THREADS) dense_tile_kernel(const WT* __restrict__ W, const float* __restrict__ X, float* __restrict__ C, int m, int b, int k) {
+__global__ void __launch_bounds__(DN_THREADS) dense_tile_kernel(const WT* __restrict__ W, const float* __restrict__ X, float* __restrict__ C, int m, int b, int k, int accumulate) {
     __shared__ float sw[DN_K][DN_TILE + 4];       // [kk][weight row]
     __shared__ float sx[DN_K][DN_TILE + 4];       // [kk][batch row]
     const int m0 = blockIdx.x * DN_TILE, b0 = blockIdx.y * DN_TILE;
@@ -64,13 +64,14 @@ __global__ void __launch_bounds__(DN_THREADS) dense_tile_kernel(const WT* __rest
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int mi = m0 + tx * 4 + j;
-            if (mi < m) C[(int64_t)bi * m + mi] = acc[i][j];
+            if (mi < m) C[(int64_t)bi * m + mi] = accumulate ? C[(int64_t)bi * m + mi] + acc[i][j] : acc[i][j];
         }
     }
 }
 
 int cc_launch_prefill_bf16(cc_device* dev, const cc_buf* w, const float* x_f32, float* out, int64_t m, int64_t k, int64_t b);   // prefill_gemm.cu
 bool cc_prefill_bf16_supported(int64_t m, int64_t k, int64_t b);
+int cc_launch_dense_tile(cc_device* dev, const cc_buf* w, const float* x, float* out, int64_t m, int64_t k, int64_t b, int accumulate);
 
 bool cc_dense_supported(int wtype, int64_t b) { return (wtype == CC_F32 || wtype == CC_BF16) && b >= 8; }
 
@@ -78,9 +79,14 @@ int cc_launch_dense(cc_device* dev, const cc_buf* w, const float* x, float* out,
     if (m == 0 || b == 0) return CC_OK;
     if (w->dtype == CC_BF16 && cc_prefill_bf16_supported(m, k, b) && ((uintptr_t)w->plane[0] & 15) == 0)
         return cc_launch_prefill_bf16(dev, w, x, out, m, k, b);
+    return cc_launch_dense_tile(dev, w, x, out, m, k, b, 0);
+}
+// the SIMT tiles whatever the sizes; accumulate != 0: out += the product
+int cc_launch_dense_tile(cc_device* dev, const cc_buf* w, const float* x, float* out, int64_t m, int64_t k, int64_t b, int accumulate) {
+    if (m == 0 || b == 0) return CC_OK;
     dim3 grid((unsigned)((m + DN_TILE - 1) / DN_TILE), (unsigned)((b + DN_TILE - 1) / DN_TILE));
-    if (w->dtype == CC_F32) dense_tile_kernel<float, false><<<grid, DN_THREADS, 0, dev->stream>>>((const float*)w->plane[0], x, out, (int)m, (int)b, (int)k);
-    else if (w->dtype == CC_BF16) dense_tile_kernel<uint16_t, true><<<grid, DN_THREADS, 0, dev->stream>>>((const uint16_t*)w->plane[0], x, out, (int)m, (int)b, (int)k);
+    if (w->dtype == CC_F32) dense_tile_kernel<float, false><<<grid, DN_THREADS, 0, dev->stream>>>((const float*)w->plane[0], x, out, (int)m, (int)b, (int)k, accumulate);
+    else if (w->dtype == CC_BF16) dense_tile_kernel<uint16_t, true><<<grid, DN_THREADS, 0, dev->stream>>>((const uint16_t*)w->plane[0], x, out, (int)m, (int)b, (int)k, accumulate);
     else return cc_fail(dev, CC_ERR_UNSUPPORTED, "dense matmul: weight type %d", w->dtype);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;

@@ -1,4 +1,4 @@
-// mixers.hpp -- mixers that more than one family's runner drives: latent attention over a ring of shared cache rows (Meresun, Papunex) and the
+// mixers.hpp -- mixers that more than one family's runner drives: latent attention over a ring of shared cache rows (Meresun, Papunex, Vadodra) and the
 // state-space mixer (Vuzinex, Papunex).  Like the runners they hold weights' handles and say in which order the tensor ops run; sizes,
 // weights and constants are filled in by the family, the sequence's state (a ring; a matrix and a convolution tail) is passed in.
 #pragma once
@@ -36,6 +36,8 @@ struct LatentAttention {
     int32_t heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0;
     int32_t window = 0;                                   // <= 0: every earlier position (the ring then holds the whole sequence)
     float scale = 1.0f, rot_mag = 1.0f, norm_eps = 0.0f;
+    int32_t pairing = CC_ROPE_NEIGHBOURS;                 // which columns of the rotated part turn together
+    bool gate_per_head = false;                           // few-row form with a gate: one number per head instead of one per output column
     CudaTensor dkv_norm, uk, uv, uk_t, uv_f32, sink, rot_freq;
 
     int64_t row() const { return (int64_t)kv_rank + rot_dim; }
@@ -76,7 +78,7 @@ struct LatentAttention {
         cc_view qv = q_src.view(), ukv = uk_t.view(), rv = ring.view(), kv{}, fq{}, nw{}, sk{};
         if (kv_src) kv = kv_src->view();
         cc_buf* b = nullptr;
-        r.check(cc_latent_query_append(r.dev, &qv, (int32_t)q_col0, &ukv, heads, rot_dim, opt_view(rot_freq, fq), rot_mag, pos0, kv_src ? &kv : nullptr, (int32_t)kv_col0, &rv,
+        r.check(cc_latent_query_append_paired(r.dev, &qv, (int32_t)q_col0, &ukv, heads, rot_dim, opt_view(rot_freq, fq), pairing, rot_mag, pos0, kv_src ? &kv : nullptr, (int32_t)kv_col0, &rv,
                                        opt_view(dkv_norm, nw), norm_eps, &b));
         CudaTensor ql = r.adopt(b, {n, (int64_t)heads * row()});
         cc_view qlv = ql.view();
@@ -88,7 +90,7 @@ struct LatentAttention {
         b = nullptr;
         if (gate_src) {
             cc_view gv = gate_src->view();
-            r.check(cc_head_project_gated(r.dev, &olv, &uvv, heads, &gv, (int32_t)gate_col0, &b));
+            r.check((gate_per_head ? cc_head_project_head_gated : cc_head_project_gated)(r.dev, &olv, &uvv, heads, &gv, (int32_t)gate_col0, &b));
         } else {
             r.check(cc_head_project(r.dev, &olv, &uvv, heads, 0, nullptr, 1.0f, 0, &b));
         }
@@ -100,12 +102,26 @@ struct LatentAttention {
         cc_view rv = ring.view(), cv = ckv.view(), nw{}, fq{};
         r.check(cc_latent_ring_append(r.dev, &rv, &cv, opt_view(dkv_norm, nw), norm_eps, kv_rank, opt_view(rot_freq, fq), rot_mag, pos0));
     }
+    // many rows: the queries in the columns q_col0 .. of src, rotated, as a tensor of their own; with kv_col0 >= 0 the tokens' cache rows as well
+    CudaTensor prepare_many(csr_runner& r, CudaTensor& ring, const CudaTensor& src, int64_t q_col0, int64_t kv_col0, int64_t pos0) const {
+        check_capacity(ring, pos0 + src.shape()[0]);
+        cc_view sv = src.view(), rv = ring.view(), fq{}, nw{};
+        cc_buf* b = nullptr;
+        r.check(cc_latent_prepare_append(r.dev, &sv, (int32_t)q_col0, heads, dim, rot_dim, opt_view(rot_freq, fq), pairing, rot_mag, pos0, kv_col0 >= 0 ? &sv : nullptr,
+                                         kv_col0 >= 0 ? (int32_t)kv_col0 : 0, &rv, opt_view(dkv_norm, nw), norm_eps, &b));
+        return r.adopt(b, {src.shape()[0], q_cols()});
+    }
     // many rows, the tokens' cache rows already in the ring; q: their raw queries (rotated in place).  -> [n, heads * vdim]
     CudaTensor attend_many(csr_runner& r, CudaTensor& ring, const CudaTensor& q, int64_t pos0) const {
+        cc_view qv = q.view(), fq{};
+        if (rot_freq.valid())
+            r.check((pairing == CC_ROPE_HALVES ? cc_rope_halves : cc_rope_pairs)(r.dev, &qv, heads, dim + rot_dim, dim, opt_view(rot_freq, fq), rot_mag, pos0));
+        return attend_rotated(r, ring, q, pos0);
+    }
+    CudaTensor attend_rotated(csr_runner& r, CudaTensor& ring, const CudaTensor& q, int64_t pos0) const {
         const int64_t n = q.shape()[0], cap = ring.shape()[0];
         check_capacity(ring, pos0 + n);
-        cc_view qv = q.view(), rv = ring.view(), fq{}, sk{};
-        if (rot_freq.valid()) r.check(cc_rope_pairs(r.dev, &qv, heads, dim + rot_dim, dim, opt_view(rot_freq, fq), rot_mag, pos0));
+        cc_view qv = q.view(), rv = ring.view(), sk{};
         // the expansion keeps the ring's row order (position p in row p % ring), so the attention reads it like the ring itself; rows no token
         // has written yet are never visible
         const int64_t rows = std::min<int64_t>(cap, pos0 + n);

@@ -224,12 +224,6 @@ template <class WT> __device__ __forceinline__ float moe_round(float v);
 template <> __device__ __forceinline__ float moe_round<float>(float v) { return v; }
 template <> __device__ __forceinline__ float moe_round<uint16_t>(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 
-// the gated unit: act(min(g, limit)) * (clamp(u, -limit, limit) + up_shift); limit <= 0 clamps nothing
-__device__ __forceinline__ float moe_glu(float g, float u, const cc_glu_params P) {
-    if (P.limit > 0.0f) { g = fminf(g, P.limit); u = fminf(fmaxf(u, -P.limit), P.limit); }
-    return act_apply(g, P.act, P.alpha) * (u + P.up_shift);
-}
-
 // one lane's share of a row's dot product with a vector in shared memory.  VEC: 16-byte pieces (4 floats or 8 bfloat16) of the row, lane-strided;
 // else element by element
 template <class WT, bool VEC> __device__ __forceinline__ float moe_dot(const WT* __restrict__ w, const float* xs, int n, int lane) {
@@ -271,7 +265,7 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(const float* __restric
     float g = wg ? moe_dot<WT, VEC>(wg + base, mg_sm, D, lane) : 0.0f, u = moe_dot<WT, VEC>(wu + base, mg_sm, D, lane);
     if (wg) g = warp_sum(g);
     u = warp_sum(u);
-    if (lane == 0) hid[(int64_t)ts * ff + r] = wg ? moe_glu(g, u, act) : act_apply(u, act.act, act.alpha);
+    if (lane == 0) hid[(int64_t)ts * ff + r] = wg ? glu_apply(g, u, act) : act_apply(u, act.act, act.alpha);
 }
 // grid (T, ceil(D / 8)), 256 threads: the CTA stages the token's top hidden rows; a warp owns one output coordinate and adds the slots in order
 template <class WT, bool VEC>
@@ -362,7 +356,7 @@ __global__ void moe_glu_bf16_kernel(const float* __restrict__ g, const float* __
     const float2 uv = *(const float2*)(u + i);
     if (g) {
         const float2 gv = *(const float2*)(g + i);
-        *(__nv_bfloat162*)(h + i) = __floats2bfloat162_rn(moe_glu(gv.x, uv.x, act), moe_glu(gv.y, uv.y, act));
+        *(__nv_bfloat162*)(h + i) = __floats2bfloat162_rn(glu_apply(gv.x, uv.x, act), glu_apply(gv.y, uv.y, act));
     } else {                                                  // a plain unit: act(u)
         *(__nv_bfloat162*)(h + i) = __floats2bfloat162_rn(act_apply(uv.x, act.act, act.alpha), act_apply(uv.y, act.act, act.alpha));
     }

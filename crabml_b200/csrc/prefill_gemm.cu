@@ -91,7 +91,8 @@ struct PgShared {
 // than it delivers (profiles/r02e: 47 % tensor pipe with MT = 1).
 template <int BLOCK_N, int MT, int FMT = 0>
 __global__ void __launch_bounds__(PG_THREADS, 1) umma_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x,
-                                                                  float* __restrict__ C, int m, int b, int k, const int* __restrict__ groups = nullptr) {
+                                                                  float* __restrict__ C, int m, int b, int k, const int* __restrict__ groups = nullptr,
+                                                                  int accumulate = 0) {
     // grouped mode (groups != nullptr; routed experts, moe.cu): groups[0] = number of tiles, then per tile {group, first row, rows, 0}.
     // Tile y multiplies rows [first, first + rows) of X with the weight rows [group * m, (group + 1) * m) of the stacked W; m is the
     // per-group row count.  Rows a tile loads beyond its own (the next group's, or zero fill) are computed and never stored.
@@ -188,7 +189,16 @@ __global__ void __launch_bounds__(PG_THREADS, 1) umma_gemm_kernel(const __grid_c
                   "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
                 : "r"(taddr));
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-            if (row < m) {
+            if (row < m && accumulate) {                                 // C += the product: the residual stream is updated where it lies
+                float old[32];
+#pragma unroll
+                for (int j = 0; j < 32; j++) old[j] = n0 + c0 + j < b ? C[(size_t)(n0 + c0 + j) * m + row] : 0.0f;
+#pragma unroll
+                for (int j = 0; j < 32; j++) {
+                    const int bi = n0 + c0 + j;
+                    if (bi < b) C[(size_t)bi * m + row] = old[j] + __uint_as_float(v[j]);
+                }
+            } else if (row < m) {
 #pragma unroll
                 for (int j = 0; j < 32; j++) {
                     const int bi = n0 + c0 + j;
@@ -299,13 +309,13 @@ bool cc_prefill_supported(int wtype, int64_t m, int64_t k, int64_t b) {
 }
 
 template <int BLOCK_N, int MT, int FMT = 0>
-static int pg_launch(cc_device* dev, const CUtensorMap& tw, const CUtensorMap& tx, float* out, int64_t m, int64_t b, int64_t k) {
+static int pg_launch(cc_device* dev, const CUtensorMap& tw, const CUtensorMap& tx, float* out, int64_t m, int64_t b, int64_t k, int accumulate = 0) {
     const size_t stage = (size_t)MT * PG_BLOCK_M * PG_BLOCK_K * 2 + (size_t)BLOCK_N * PG_BLOCK_K * 2;
     const int stages = stage * PG_STAGES <= 200 * 1024 ? PG_STAGES : 3;
     const size_t smem = (size_t)stages * stage + 1024;
     CC_CUDA(dev, cudaFuncSetAttribute(umma_gemm_kernel<BLOCK_N, MT, FMT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     dim3 grid((unsigned)((m + PG_BLOCK_M * MT - 1) / (PG_BLOCK_M * MT)), (unsigned)((b + BLOCK_N - 1) / BLOCK_N));
-    umma_gemm_kernel<BLOCK_N, MT, FMT><<<grid, PG_THREADS, smem, dev->stream>>>(tw, tx, out, (int)m, (int)b, (int)k);
+    umma_gemm_kernel<BLOCK_N, MT, FMT><<<grid, PG_THREADS, smem, dev->stream>>>(tw, tx, out, (int)m, (int)b, (int)k, nullptr, accumulate);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
@@ -375,6 +385,27 @@ bool cc_prefill_bf16_supported(int64_t m, int64_t k, int64_t b) {
     static const bool off = getenv("CRABML_PREFILL_OFF") != nullptr;
     return !off && b >= 32 && m >= 1 && k >= PG_BLOCK_K && k % PG_BLOCK_K == 0;
 }
+// the device's scratch for a bfloat16 operand [b][k]; a caller that makes the operand itself fills it and calls the launch below
+int cc_prefill_bf16_operand(cc_device* dev, int64_t b, int64_t k, void** out) {
+    PgScratch* s = pg_scratch(dev);
+    int rc = pg_ensure(dev, &s->x, &s->x_bytes, (size_t)b * k * 2);
+    *out = s->x;
+    return rc;
+}
+// the product over the operand in that scratch; accumulate != 0: out += it
+int cc_launch_prefill_bf16_operand(cc_device* dev, const cc_buf* w, float* out, int64_t m, int64_t k, int64_t b, int accumulate) {
+    PgScratch* s = pg_scratch(dev);
+    const int block_n = b >= 192 ? 256 : b >= 96 ? 128 : 64;
+    CUtensorMap tw, tx;
+    int rc = pg_make_tmap(dev, &tw, w->plane[0], m, k, PG_BLOCK_M, true);
+    if (rc) return rc;
+    rc = pg_make_tmap(dev, &tx, s->x, b, k, block_n, true);
+    if (rc) return rc;
+    const bool mt2 = m >= 512;
+    if (block_n == 256) return mt2 ? pg_launch<256, 2, 1>(dev, tw, tx, out, m, b, k, accumulate) : pg_launch<256, 1, 1>(dev, tw, tx, out, m, b, k, accumulate);
+    if (block_n == 128) return mt2 ? pg_launch<128, 2, 1>(dev, tw, tx, out, m, b, k, accumulate) : pg_launch<128, 1, 1>(dev, tw, tx, out, m, b, k, accumulate);
+    return mt2 ? pg_launch<64, 2, 1>(dev, tw, tx, out, m, b, k, accumulate) : pg_launch<64, 1, 1>(dev, tw, tx, out, m, b, k, accumulate);
+}
 int cc_launch_prefill_bf16_act(cc_device* dev, const cc_buf* w, const float* x_f32, int act, float* out, int64_t m, int64_t k, int64_t b) {
     PgScratch* s = pg_scratch(dev);
     int rc = pg_ensure(dev, &s->x, &s->x_bytes, (size_t)b * k * 2);
@@ -382,16 +413,7 @@ int cc_launch_prefill_bf16_act(cc_device* dev, const cc_buf* w, const float* x_f
     const int64_t na = b * k;
     act_f32_to_bf16_kernel<<<(unsigned)((na / 2 + 255) / 256), 256, 0, dev->stream>>>(x_f32, na, (__nv_bfloat16*)s->x, act);
     CC_LAUNCH_CHECK(dev);
-    const int block_n = b >= 192 ? 256 : b >= 96 ? 128 : 64;
-    CUtensorMap tw, tx;
-    rc = pg_make_tmap(dev, &tw, w->plane[0], m, k, PG_BLOCK_M, true);
-    if (rc) return rc;
-    rc = pg_make_tmap(dev, &tx, s->x, b, k, block_n, true);
-    if (rc) return rc;
-    const bool mt2 = m >= 512;
-    if (block_n == 256) return mt2 ? pg_launch<256, 2, 1>(dev, tw, tx, out, m, b, k) : pg_launch<256, 1, 1>(dev, tw, tx, out, m, b, k);
-    if (block_n == 128) return mt2 ? pg_launch<128, 2, 1>(dev, tw, tx, out, m, b, k) : pg_launch<128, 1, 1>(dev, tw, tx, out, m, b, k);
-    return mt2 ? pg_launch<64, 2, 1>(dev, tw, tx, out, m, b, k) : pg_launch<64, 1, 1>(dev, tw, tx, out, m, b, k);
+    return cc_launch_prefill_bf16_operand(dev, w, out, m, k, b, 0);
 }
 
 int cc_launch_prefill_bf16(cc_device* dev, const cc_buf* w, const float* x_f32, float* out, int64_t m, int64_t k, int64_t b) {

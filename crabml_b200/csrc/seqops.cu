@@ -11,6 +11,7 @@
 #include "../../include/crabml_seqops.h"
 #include "act.cuh"
 #include "capi_checks.cuh"
+#include "layer_norm.cuh"
 
 #define SEQ_ENTER(dev, what)                                                                                          \
     if (!(dev)) return CC_ERR_ARG;                                                                                    \
@@ -268,20 +269,30 @@ extern "C" CC_API int cc_scaled_sum_accumulate(cc_device* dev, const cc_view* ds
     return CC_OK;
 }
 // one gate number per (row, head): one thread per element
-__global__ void head_gate_kernel(float* __restrict__ x, const float* __restrict__ g, int64_t n, int hs, int act) {
+__global__ void head_gate_kernel(float* __restrict__ x, const float* __restrict__ g, int64_t n, int hs, int heads, int64_t grs, int act) {
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) x[i] *= seq_act(g[i / hs], act);
+    if (i >= n) return;
+    const int64_t u = i / hs, t = u / heads;
+    x[i] *= seq_act(g[t * grs + (u - t * heads)], act);
+}
+// gate numbers in the columns col0 .. col0 + n_heads of g's rows
+static int head_gate_impl(cc_device* dev, const cc_view* x, const cc_view* g, int32_t col0, int32_t n_heads, int32_t act) {
+    SEQ_F32(dev, x, "head_gate x"); SEQ_ROWS(dev, g, "head_gate g");
+    CC_REQUIRE(dev, x->ndim == 2 && n_heads > 0 && x->shape[1] % n_heads == 0 && g->shape[0] == x->shape[0] && col0 >= 0 && (int64_t)col0 + n_heads <= g->shape[1],
+               "head_gate: x must be [rows, heads * head_size] and g hold %d columns from column %d on", n_heads, col0);
+    const int64_t n = view_len(x);
+    if (!n) return CC_OK;
+    head_gate_kernel<<<(unsigned)((n + 255) / 256), 256, 0, dev->stream>>>(fptr(x), fptr(g) + col0, n, (int)(x->shape[1] / n_heads), n_heads, g->strides[0], act);
+    CC_LAUNCH_CHECK(dev);
+    return CC_OK;
 }
 extern "C" CC_API int cc_head_gate(cc_device* dev, const cc_view* x, const cc_view* g, int32_t n_heads, int32_t act) {
     SEQ_ENTER(dev, "head_gate");
-    SEQ_F32(dev, x, "head_gate x"); SEQ_F32(dev, g, "head_gate g");
-    CC_REQUIRE(dev, x->ndim == 2 && n_heads > 0 && x->shape[1] % n_heads == 0 && view_len(g) == x->shape[0] * n_heads,
-               "head_gate: x must be [rows, heads * head_size] and g [rows, heads]");
-    const int64_t n = view_len(x);
-    if (!n) return CC_OK;
-    head_gate_kernel<<<(unsigned)((n + 255) / 256), 256, 0, dev->stream>>>(fptr(x), fptr(g), n, (int)(x->shape[1] / n_heads), act);
-    CC_LAUNCH_CHECK(dev);
-    return CC_OK;
+    return head_gate_impl(dev, x, g, 0, n_heads, act);
+}
+extern "C" CC_API int cc_head_gate_cols(cc_device* dev, const cc_view* x, const cc_view* gate_src, int32_t gate_col0, int32_t n_heads, int32_t act) {
+    SEQ_ENTER(dev, "head_gate");
+    return head_gate_impl(dev, x, gate_src, gate_col0, n_heads, act);
 }
 // out = [a | b] row by row: one thread per element of out
 __global__ void concat_cols_kernel(const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ out, int64_t n, int ca, int cb) {
@@ -1213,52 +1224,12 @@ extern "C" CC_API int cc_group_rms_norm(cc_device* dev, const cc_view* dst, cons
 }
 
 // ---- layer norm with weight and bias ------------------------------------------------------------------------------------------------------
-// one CTA per row: a thread keeps its (up to LN_KEEP) elements of the row in registers, so the row is read once; the mean first
-// (thread-strided partial sums, the butterfly, then the warps' sums in warp order), then the mean of the squared deviations from it in the same
-// order, then the scaled write.  The order depends on the row's length alone.
+// one CTA per row (layer_norm.cuh)
 #define LN_THREADS 256
-#define LN_KEEP 8
-__device__ __forceinline__ float ln_block_sum(float v, float* red) {
-    v = warp_sum(v);
-    __syncthreads();                                         // red may still be read from the sum before
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-    __syncthreads();
-    float t = 0.0f;
-#pragma unroll
-    for (int w = 0; w < LN_THREADS / 32; w++) t += red[w];
-    return t;
-}
 __global__ void __launch_bounds__(LN_THREADS) layer_norm_kernel(float* dst, const float* x, const float* __restrict__ w, const float* __restrict__ b, int cols, float eps) {
     __shared__ float red[LN_THREADS / 32];
-    const float* xr = x + (int64_t)blockIdx.x * cols;
     float* dr = dst + (int64_t)blockIdx.x * cols;
-    float keep[LN_KEEP];
-    float s = 0.0f;
-#pragma unroll
-    for (int e = 0; e < LN_KEEP; e++) {
-        const int c = threadIdx.x + e * LN_THREADS;
-        keep[e] = c < cols ? xr[c] : 0.0f;
-        s += keep[e];
-    }
-    for (int c = threadIdx.x + LN_KEEP * LN_THREADS; c < cols; c += LN_THREADS) s += xr[c];
-    const float mean = ln_block_sum(s, red) / (float)cols;
-    float ss = 0.0f;
-#pragma unroll
-    for (int e = 0; e < LN_KEEP; e++) {
-        const int c = threadIdx.x + e * LN_THREADS;
-        const float d = keep[e] - mean;
-        if (c < cols) ss = fmaf(d, d, ss);
-    }
-    for (int c = threadIdx.x + LN_KEEP * LN_THREADS; c < cols; c += LN_THREADS) { const float d = xr[c] - mean; ss = fmaf(d, d, ss); }
-    const float inv = 1.0f / sqrtf(ln_block_sum(ss, red) / (float)cols + eps);
-    // a row wider than the registers hold is read again here, before any of it is overwritten by another thread: dst may be x, and thread t only
-    // ever touches columns t, t + 256, ...
-#pragma unroll
-    for (int e = 0; e < LN_KEEP; e++) {
-        const int c = threadIdx.x + e * LN_THREADS;
-        if (c < cols) { const float v = (keep[e] - mean) * inv * w[c]; dr[c] = b ? v + b[c] : v; }
-    }
-    for (int c = threadIdx.x + LN_KEEP * LN_THREADS; c < cols; c += LN_THREADS) { const float v = (xr[c] - mean) * inv * w[c]; dr[c] = b ? v + b[c] : v; }
+    layer_norm_row<LN_THREADS>(x + (int64_t)blockIdx.x * cols, w, b, cols, eps, red, [&](int c, float v) { dr[c] = v; });
 }
 extern "C" CC_API int cc_layer_norm(cc_device* dev, const cc_view* dst, const cc_view* x, const cc_view* w, const cc_view* b, float eps) {
     SEQ_ENTER(dev, "layer_norm");
@@ -1385,8 +1356,10 @@ static int rope_table_impl(cc_device* dev, const cc_view* x, int32_t n_heads, in
 
 // ---- queries and keys from projection to cache in one pass ---------------------------------------------------------------------------------
 struct QkPrepArgs {
-    float *q, *kring, *vring;
-    const float *k, *v, *qw, *kw, *freq;
+    const float *q, *k, *v;                                 // row t of the raw operands at q + t * qrs, k + t * krs, v + t * vrs
+    float *qo, *kring, *vring;                              // qo: [T, H * dk], may be q itself
+    int64_t qrs, krs, vrs;
+    const float *qw, *kw, *freq;
     int H, G, dk, dv, ring, norm, half, step, gap, off;      // pair i of a head: columns off + i * step and off + i * step + gap
     float eps, mag;
     int64_t pos0;
@@ -1401,8 +1374,9 @@ __global__ void __launch_bounds__(QKP_THREADS) qk_prepare_kernel(QkPrepArgs a) {
     float* inv = qkp_sm;
     float* red = qkp_sm + a.H + a.G;
     const int t = blockIdx.x, lane = threadIdx.x & 31, w = threadIdx.x >> 5;
-    float* qr = a.q + (int64_t)t * a.H * a.dk;
-    const float* kr = a.k + (int64_t)t * a.G * a.dk;
+    const float* qr = a.q + t * a.qrs;
+    const float* kr = a.k + t * a.krs;
+    float* qo = a.qo + (int64_t)t * a.H * a.dk;
     const int units = a.H + a.G;
     if (a.norm == CC_QK_NORM_HEAD) {
         for (int u = w; u < units; u += QKP_THREADS / 32) {
@@ -1439,7 +1413,7 @@ __global__ void __launch_bounds__(QKP_THREADS) qk_prepare_kernel(QkPrepArgs a) {
         const bool is_q = u < a.H;
         const int ul = is_q ? u : u - a.H;
         const float* src = is_q ? qr + u * a.dk : kr + ul * a.dk;
-        float* dst = is_q ? qr + u * a.dk : a.kring + (row * a.G + ul) * a.dk;
+        float* dst = is_q ? qo + u * a.dk : a.kring + (row * a.G + ul) * a.dk;
         const float* wt = is_q ? a.qw : a.kw;
         if (wt && a.norm == CC_QK_NORM_ROW) wt += ul * a.dk;
         const float f = inv[u];
@@ -1461,21 +1435,16 @@ __global__ void __launch_bounds__(QKP_THREADS) qk_prepare_kernel(QkPrepArgs a) {
             dst[c] = x0;
         }
     }
-    const float* vr = a.v + (int64_t)t * a.G * a.dv;
+    const float* vr = a.v + t * a.vrs;
     float* vd = a.vring + row * a.G * a.dv;
     for (int c = threadIdx.x; c < a.G * a.dv; c += QKP_THREADS) vd[c] = vr[c];
 }
-extern "C" CC_API int cc_qk_prepare_append(cc_device* dev, const cc_view* q, const cc_view* k, const cc_view* v, const cc_view* kring, const cc_view* vring, int32_t qk_norm,
-                                           const cc_view* q_w, const cc_view* k_w, float eps, const cc_view* freq, int32_t pairing, int32_t offset, float mag, int64_t pos0,
-                                           int32_t H, int32_t G, int32_t dk, int32_t dv) {
-    SEQ_ENTER(dev, "qk_prepare_append");
-    SEQ_F32(dev, q, "qk_prepare_append q"); SEQ_F32(dev, k, "qk_prepare_append k"); SEQ_F32(dev, v, "qk_prepare_append v");
+static int qk_prepare_impl(cc_device* dev, QkPrepArgs a, int64_t T, const cc_view* kring, const cc_view* vring, int32_t qk_norm, const cc_view* q_w, const cc_view* k_w, float eps,
+                           const cc_view* freq, int32_t pairing, int32_t offset, float mag, int64_t pos0, int32_t H, int32_t G, int32_t dk, int32_t dv) {
     SEQ_F32(dev, kring, "qk_prepare_append kring"); SEQ_F32(dev, vring, "qk_prepare_append vring");
-    CC_REQUIRE(dev, H > 0 && G > 0 && dk > 0 && dv > 0 && q->ndim == 2 && kring->ndim == 2 && pos0 >= 0 && qk_norm >= CC_QK_NORM_NONE && qk_norm <= CC_QK_NORM_ROW,
-               "qk_prepare_append: bad arguments");
-    const int64_t T = q->shape[0], ring = kring->shape[0];
-    CC_REQUIRE(dev, view_len(q) == T * H * dk && view_len(k) == T * G * dk && view_len(v) == T * G * dv && view_len(kring) == ring * G * dk && view_len(vring) == ring * G * dv,
-               "qk_prepare_append: operand sizes do not fit heads=%d kv=%d dk=%d dv=%d", H, G, dk, dv);
+    CC_REQUIRE(dev, kring->ndim == 2 && pos0 >= 0 && qk_norm >= CC_QK_NORM_NONE && qk_norm <= CC_QK_NORM_ROW, "qk_prepare_append: bad arguments");
+    const int64_t ring = kring->shape[0];
+    CC_REQUIRE(dev, view_len(kring) == ring * G * dk && view_len(vring) == ring * G * dv, "qk_prepare_append: the rings do not fit kv=%d dk=%d dv=%d", G, dk, dv);
     CC_REQUIRE(dev, T <= ring, "qk_prepare_append: %lld tokens do not fit a ring of %lld", (long long)T, (long long)ring);
     const int64_t wq = qk_norm == CC_QK_NORM_ROW ? (int64_t)H * dk : dk, wk = qk_norm == CC_QK_NORM_ROW ? (int64_t)G * dk : dk;
     if (q_w) { SEQ_F32(dev, q_w, "qk_prepare_append q_w"); CC_REQUIRE(dev, qk_norm != CC_QK_NORM_NONE && view_len(q_w) == wq, "qk_prepare_append: q_w must have %lld elements", (long long)wq); }
@@ -1488,8 +1457,7 @@ extern "C" CC_API int cc_qk_prepare_append(cc_device* dev, const cc_view* q, con
                    (long long)half, offset, dk);
     }
     if (T == 0) return CC_OK;
-    QkPrepArgs a{};
-    a.q = fptr(q); a.k = fptr(k); a.v = fptr(v); a.kring = fptr(kring); a.vring = fptr(vring); a.qw = q_w ? fptr(q_w) : nullptr; a.kw = k_w ? fptr(k_w) : nullptr;
+    a.kring = fptr(kring); a.vring = fptr(vring); a.qw = q_w ? fptr(q_w) : nullptr; a.kw = k_w ? fptr(k_w) : nullptr;
     a.freq = freq ? fptr(freq) : nullptr; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.ring = (int)ring; a.norm = qk_norm; a.half = (int)half; a.off = offset;
     a.step = pairing == CC_ROPE_HALVES ? 1 : 2; a.gap = pairing == CC_ROPE_HALVES ? (int)half : 1; a.eps = eps; a.mag = mag; a.pos0 = pos0;
     const size_t smem = (size_t)(H + G + QKP_THREADS / 32) * 4;
@@ -1498,6 +1466,38 @@ extern "C" CC_API int cc_qk_prepare_append(cc_device* dev, const cc_view* q, con
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
+extern "C" CC_API int cc_qk_prepare_append_cols(cc_device* dev, const cc_view* src, int32_t q_col0, int32_t k_col0, int32_t v_col0, const cc_view* kring, const cc_view* vring,
+                                                int32_t qk_norm, const cc_view* q_w, const cc_view* k_w, float eps, const cc_view* freq, int32_t pairing, int32_t offset, float mag,
+                                                int64_t pos0, int32_t H, int32_t G, int32_t dk, int32_t dv, cc_buf** out) {
+    SEQ_ENTER(dev, "qk_prepare_append_cols");
+    if (!out) return cc_fail(dev, CC_ERR_ARG, "qk_prepare_append_cols: out is NULL");
+    SEQ_ROWS(dev, src, "qk_prepare_append_cols src");
+    CC_REQUIRE(dev, H > 0 && G > 0 && dk > 0 && dv > 0, "qk_prepare_append_cols: bad arguments");
+    const int64_t T = src->shape[0], cols = src->shape[1];
+    CC_REQUIRE(dev, q_col0 >= 0 && k_col0 >= 0 && v_col0 >= 0 && q_col0 + (int64_t)H * dk <= cols && k_col0 + (int64_t)G * dk <= cols && v_col0 + (int64_t)G * dv <= cols,
+               "qk_prepare_append_cols: columns %d / %d / %d of %lld do not fit heads=%d kv=%d dk=%d dv=%d", q_col0, k_col0, v_col0, (long long)cols, H, G, dk, dv);
+    cc_buf* o = nullptr;
+    int rc = cc_new_activation(dev, T * H * dk, CC_F32, false, &o);
+    if (rc) return rc;
+    QkPrepArgs a{};
+    a.q = fptr(src) + q_col0; a.k = fptr(src) + k_col0; a.v = fptr(src) + v_col0; a.qo = (float*)o->base; a.qrs = a.krs = a.vrs = src->strides[0];
+    rc = qk_prepare_impl(dev, a, T, kring, vring, qk_norm, q_w, k_w, eps, freq, pairing, offset, mag, pos0, H, G, dk, dv);
+    if (rc) { cc_tensor_release(o); return rc; }
+    *out = o;
+    return CC_OK;
+}
+extern "C" CC_API int cc_qk_prepare_append(cc_device* dev, const cc_view* q, const cc_view* k, const cc_view* v, const cc_view* kring, const cc_view* vring, int32_t qk_norm,
+                                           const cc_view* q_w, const cc_view* k_w, float eps, const cc_view* freq, int32_t pairing, int32_t offset, float mag, int64_t pos0,
+                                           int32_t H, int32_t G, int32_t dk, int32_t dv) {
+    SEQ_ENTER(dev, "qk_prepare_append");
+    SEQ_F32(dev, q, "qk_prepare_append q"); SEQ_F32(dev, k, "qk_prepare_append k"); SEQ_F32(dev, v, "qk_prepare_append v");
+    CC_REQUIRE(dev, H > 0 && G > 0 && dk > 0 && dv > 0 && q->ndim == 2, "qk_prepare_append: bad arguments");
+    const int64_t T = q->shape[0];
+    CC_REQUIRE(dev, view_len(q) == T * H * dk && view_len(k) == T * G * dk && view_len(v) == T * G * dv, "qk_prepare_append: operand sizes do not fit heads=%d kv=%d dk=%d dv=%d", H, G, dk, dv);
+    QkPrepArgs a{};
+    a.q = fptr(q); a.k = fptr(k); a.v = fptr(v); a.qo = fptr(q); a.qrs = (int64_t)H * dk; a.krs = (int64_t)G * dk; a.vrs = (int64_t)G * dv;
+    return qk_prepare_impl(dev, a, T, kring, vring, qk_norm, q_w, k_w, eps, freq, pairing, offset, mag, pos0, H, G, dk, dv);
+}
 
 // ---- latent key/value cache ------------------------------------------------------------------------------------------------------------------
 // one warp per token: the first `rank` columns are RMS-normalised and weighted, the pairs of the next columns rotated, the rest copied
@@ -1505,7 +1505,7 @@ struct LatAppend {
     float* ring;                  // NULL: nothing to append
     const float *ckv, *nw, *freq; // row t of the raw rows at ckv + t * rs
     int64_t rs, pos0;
-    int ring_rows, rank, rest, half;
+    int ring_rows, rank, rest, half, step, gap;      // pair i of the rotated part: its columns step * i and step * i + gap
     float eps, mag;
 };
 __device__ __forceinline__ void latent_append_row(const LatAppend& a, int t, int lane) {
@@ -1521,8 +1521,9 @@ __device__ __forceinline__ void latent_append_row(const LatAppend& a, int t, int
     for (int c = lane; c < rank; c += 32) dst[c] = src[c] * inv * (nw ? nw[c] : 1.0f);
     for (int i = lane; i < half; i += 32) {
         float ou, ov;
-        rotate_pair(src[rank + 2 * i], src[rank + 2 * i + 1], (float)(pos0 + t), freq[i], mag, ou, ov);
-        dst[rank + 2 * i] = ou; dst[rank + 2 * i + 1] = ov;
+        const int c = rank + a.step * i;
+        rotate_pair(src[c], src[c + a.gap], (float)(pos0 + t), freq[i], mag, ou, ov);
+        dst[c] = ou; dst[c + a.gap] = ov;
     }
     for (int c = rank + 2 * half + lane; c < cols; c += 32) dst[c] = src[c];
 }
@@ -1542,7 +1543,7 @@ extern "C" CC_API int cc_latent_ring_append(cc_device* dev, const cc_view* ring,
                (long long)half, (long long)cols);
     CC_REQUIRE(dev, T <= ring->shape[0], "latent_ring_append: %lld tokens do not fit a ring of %lld", (long long)T, (long long)ring->shape[0]);
     if (T == 0) return CC_OK;
-    const LatAppend a = {fptr(ring), fptr(ckv), norm_w ? fptr(norm_w) : nullptr, freq ? fptr(freq) : nullptr, cols, pos0, (int)ring->shape[0], rank, (int)(cols - rank), (int)half, eps, mag};
+    const LatAppend a = {fptr(ring), fptr(ckv), norm_w ? fptr(norm_w) : nullptr, freq ? fptr(freq) : nullptr, cols, pos0, (int)ring->shape[0], rank, (int)(cols - rank), (int)half, 2, 1, eps, mag};
     latent_ring_append_kernel<<<(unsigned)((T + 7) / 8), 256, 0, dev->stream>>>(a, (int)T);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
@@ -1554,8 +1555,8 @@ struct HpArgs {
     const float *x, *W;           // token t's row at x + t * xrs, head h's inputs at + h * (n_in + rest)
     float* out;
     int64_t xrs, grs, pos0;
-    const float *freq, *gate;     // gate (rest == 0 only): output (t, h, v) is multiplied by sigmoid(gate[t * grs + h * n_out + v]); NULL: not gated
-    int T, H, n_in, rest, n_out, half;
+    const float *freq, *gate;     // gate (rest == 0 only): output (t, h, v) is multiplied by sigmoid(gate[t * grs + h * ghs + v * gvs]); NULL: not gated
+    int T, H, n_in, rest, n_out, half, step, gap, ghs, gvs;
     float mag;
     LatAppend app;                // app.ring != NULL: the grid has one more z plane, whose CTAs of head 0 write the tokens' cache rows
 };
@@ -1580,9 +1581,9 @@ __global__ void __launch_bounds__(128) head_project_kernel(HpArgs a) {
         for (int i = threadIdx.x; i < HP_TOK * half; i += 128) {
             const int tt = i / half, p = i - tt * half;
             if (t0 + tt >= T) continue;
-            const float* src = a.x + (t0 + tt) * a.xrs + h * xs + n_in + 2 * p;
-            float* dst = a.out + ((int64_t)(t0 + tt) * H + h) * os + n_out + 2 * p;
-            rotate_pair(src[0], src[1], (float)(a.pos0 + t0 + tt), a.freq[p], a.mag, dst[0], dst[1]);
+            const float* src = a.x + (t0 + tt) * a.xrs + h * xs + n_in + a.step * p;
+            float* dst = a.out + ((int64_t)(t0 + tt) * H + h) * os + n_out + a.step * p;
+            rotate_pair(src[0], src[a.gap], (float)(a.pos0 + t0 + tt), a.freq[p], a.mag, dst[0], dst[a.gap]);
         }
         const int plain = rest - 2 * half;
         for (int i = threadIdx.x; i < HP_TOK * plain; i += 128) {
@@ -1606,7 +1607,7 @@ __global__ void __launch_bounds__(128) head_project_kernel(HpArgs a) {
     for (int tt = 0; tt < HP_TOK; tt++) {
         float sum = warp_sum(acc[tt]);
         if (lane != 0 || t0 + tt >= T) continue;
-        if (a.gate) sum *= seq_sigmoid(a.gate[(t0 + tt) * a.grs + h * n_out + v]);
+        if (a.gate) sum *= seq_sigmoid(a.gate[(t0 + tt) * a.grs + h * a.ghs + v * a.gvs]);
         a.out[((int64_t)(t0 + tt) * H + h) * os + v] = sum;
     }
 }
@@ -1691,18 +1692,27 @@ extern "C" CC_API int cc_head_project(cc_device* dev, const cc_view* x, const cc
     }
     HpArgs a{};
     a.x = fptr(x); a.W = fptr(w); a.out = (float*)o->base; a.xrs = x->shape[1]; a.pos0 = pos0; a.freq = freq ? fptr(freq) : nullptr; a.half = freq ? (int)view_len(freq) : 0; a.mag = mag;
-    a.T = (int)T; a.H = n_heads; a.n_in = (int)n_in; a.rest = rest; a.n_out = (int)n_out;
+    a.T = (int)T; a.H = n_heads; a.n_in = (int)n_in; a.rest = rest; a.n_out = (int)n_out; a.step = 2; a.gap = 1;
     return head_project_few(dev, a);
 }
+static int head_project_gated_impl(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, bool per_head, cc_buf** out);
 extern "C" CC_API int cc_head_project_gated(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, cc_buf** out) {
+    return head_project_gated_impl(dev, x, w, n_heads, gate_src, gate_col0, false, out);
+}
+extern "C" CC_API int cc_head_project_head_gated(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, cc_buf** out) {
+    return head_project_gated_impl(dev, x, w, n_heads, gate_src, gate_col0, true, out);
+}
+// per_head: one gate number per head instead of one per output column
+static int head_project_gated_impl(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, bool per_head, cc_buf** out) {
     SEQ_ENTER(dev, "head_project_gated");
     if (!out) return cc_fail(dev, CC_ERR_ARG, "head_project_gated: out is NULL");
     SEQ_F32(dev, x, "head_project_gated x"); SEQ_F32(dev, w, "head_project_gated w"); SEQ_ROWS(dev, gate_src, "head_project_gated gate");
     CC_REQUIRE(dev, x->ndim == 2 && w->ndim == 2 && n_heads > 0 && w->shape[0] % n_heads == 0 && x->shape[1] == (int64_t)n_heads * w->shape[1],
                "head_project_gated: x must be [T, heads * n_in] and w [heads * n_out, n_in]");
     const int64_t T = x->shape[0];
-    CC_REQUIRE(dev, gate_src->shape[0] == T && gate_col0 >= 0 && gate_col0 + w->shape[0] <= gate_src->shape[1], "head_project_gated: the gate needs %lld columns from column %d on",
-               (long long)w->shape[0], gate_col0);
+    const int64_t gates = per_head ? n_heads : w->shape[0];
+    CC_REQUIRE(dev, gate_src->shape[0] == T && gate_col0 >= 0 && gate_col0 + gates <= gate_src->shape[1], "head_project_gated: the gate needs %lld columns from column %d on",
+               (long long)gates, gate_col0);
     cc_buf* o = nullptr;
     int rc = cc_new_activation(dev, T * w->shape[0], CC_F32, false, &o);
     if (rc) return rc;
@@ -1711,11 +1721,18 @@ extern "C" CC_API int cc_head_project_gated(cc_device* dev, const cc_view* x, co
     HpArgs a{};
     a.x = fptr(x); a.W = fptr(w); a.out = (float*)o->base; a.xrs = x->shape[1]; a.gate = fptr(gate_src) + gate_col0; a.grs = gate_src->strides[0]; a.mag = 1.0f;
     a.T = (int)T; a.H = n_heads; a.n_in = (int)w->shape[1]; a.n_out = (int)(w->shape[0] / n_heads);
+    a.ghs = per_head ? 1 : a.n_out; a.gvs = per_head ? 0 : 1;
     return head_project_few(dev, a);
 }
 extern "C" CC_API int cc_latent_query_append(cc_device* dev, const cc_view* q_src, int32_t q_col0, const cc_view* uk_t, int32_t n_heads, int32_t rest, const cc_view* freq, float mag,
                                              int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps, cc_buf** out) {
+    return cc_latent_query_append_paired(dev, q_src, q_col0, uk_t, n_heads, rest, freq, CC_ROPE_NEIGHBOURS, mag, pos0, kv_src, kv_col0, ring, norm_w, eps, out);
+}
+extern "C" CC_API int cc_latent_query_append_paired(cc_device* dev, const cc_view* q_src, int32_t q_col0, const cc_view* uk_t, int32_t n_heads, int32_t rest, const cc_view* freq,
+                                                    int32_t pairing, float mag, int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w,
+                                                    float eps, cc_buf** out) {
     SEQ_ENTER(dev, "latent_query_append");
+    CC_REQUIRE(dev, pairing == CC_ROPE_NEIGHBOURS || pairing == CC_ROPE_HALVES, "latent_query_append: unknown pairing %d", pairing);
     if (!out) return cc_fail(dev, CC_ERR_ARG, "latent_query_append: out is NULL");
     SEQ_ROWS(dev, q_src, "latent_query_append q"); SEQ_F32(dev, uk_t, "latent_query_append uk_t");
     CC_REQUIRE(dev, uk_t->ndim == 2 && n_heads > 0 && rest >= 0 && uk_t->shape[0] % n_heads == 0 && pos0 >= 0, "latent_query_append: bad arguments");
@@ -1724,13 +1741,14 @@ extern "C" CC_API int cc_latent_query_append(cc_device* dev, const cc_view* q_sr
                (long long)(n_heads * (dim + rest)), q_col0);
     if (freq) { SEQ_F32(dev, freq, "latent_query_append freq"); CC_REQUIRE(dev, 2 * view_len(freq) <= rest, "latent_query_append: more rotated pairs than carried columns"); }
     HpArgs a{};
+    const int half = freq ? (int)view_len(freq) : 0, step = pairing == CC_ROPE_HALVES ? 1 : 2, gap = pairing == CC_ROPE_HALVES ? half : 1;
     if (kv_src) {
         SEQ_ROWS(dev, kv_src, "latent_query_append kv"); SEQ_F32(dev, ring, "latent_query_append ring");
         if (norm_w) { SEQ_F32(dev, norm_w, "latent_query_append norm_w"); CC_REQUIRE(dev, view_len(norm_w) == rank, "latent_query_append: norm_w must have %lld elements", (long long)rank); }
         CC_REQUIRE(dev, ring->ndim == 2 && ring->shape[1] == rank + rest && T <= ring->shape[0] && kv_src->shape[0] == T && kv_col0 >= 0 && kv_col0 + rank + rest <= kv_src->shape[1],
                    "latent_query_append: ring rows have rank + rest columns and so have the raw rows from column %d on", kv_col0);
         a.app = {fptr(ring), fptr(kv_src) + kv_col0, norm_w ? fptr(norm_w) : nullptr, freq ? fptr(freq) : nullptr, kv_src->strides[0], pos0, (int)ring->shape[0], (int)rank, rest,
-                 freq ? (int)view_len(freq) : 0, eps, mag};
+                 half, step, gap, eps, mag};
     }
     cc_buf* o = nullptr;
     int rc = cc_new_activation(dev, T * n_heads * (rank + rest), CC_F32, false, &o);
@@ -1738,8 +1756,61 @@ extern "C" CC_API int cc_latent_query_append(cc_device* dev, const cc_view* q_sr
     *out = o;
     if (T == 0) return CC_OK;
     a.x = fptr(q_src) + q_col0; a.W = fptr(uk_t); a.out = (float*)o->base; a.xrs = q_src->strides[0]; a.pos0 = pos0; a.freq = freq ? fptr(freq) : nullptr;
-    a.half = freq ? (int)view_len(freq) : 0; a.mag = mag; a.T = (int)T; a.H = n_heads; a.n_in = (int)dim; a.rest = rest; a.n_out = (int)rank;
+    a.half = half; a.step = step; a.gap = gap; a.mag = mag; a.T = (int)T; a.H = n_heads; a.n_in = (int)dim; a.rest = rest; a.n_out = (int)rank;
     return head_project_few(dev, a);
+}
+// the same for a pass of many rows, whose queries are not folded: one CTA per token copies the queries out of their columns, rotating the last
+// `rest` columns of every head on the way (a pair by the thread of its first column), and warp 0 writes the token's cache row
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const float* __restrict__ q, int64_t qrs, float* __restrict__ out, int H, int dim, LatAppend a) {
+    const int t = blockIdx.x, hs = dim + a.rest;
+    const float* qr = q + t * qrs;
+    float* o = out + (int64_t)t * H * hs;
+    for (int idx = threadIdx.x; idx < H * hs; idx += 256) {
+        const int rel = idx % hs - dim;
+        int pair = -1;                               // index of the pair this thread owns, -2: the pair's second column
+        if (rel >= 0 && rel < 2 * a.half) {
+            if (a.step == 1) pair = rel < a.half ? rel : -2;
+            else pair = (rel & 1) ? -2 : rel >> 1;
+        }
+        if (pair == -2) continue;
+        if (pair >= 0) {
+            float ou, ov;
+            rotate_pair(qr[idx], qr[idx + a.gap], (float)(a.pos0 + t), a.freq[pair], a.mag, ou, ov);
+            o[idx] = ou; o[idx + a.gap] = ov;
+        } else {
+            o[idx] = qr[idx];
+        }
+    }
+    if (a.ring && threadIdx.x < 32) latent_append_row(a, t, threadIdx.x);
+}
+extern "C" CC_API int cc_latent_prepare_append(cc_device* dev, const cc_view* q_src, int32_t q_col0, int32_t n_heads, int32_t dim, int32_t rest, const cc_view* freq, int32_t pairing,
+                                               float mag, int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps, cc_buf** out) {
+    SEQ_ENTER(dev, "latent_prepare_append");
+    if (!out) return cc_fail(dev, CC_ERR_ARG, "latent_prepare_append: out is NULL");
+    SEQ_ROWS(dev, q_src, "latent_prepare_append q");
+    CC_REQUIRE(dev, n_heads > 0 && dim > 0 && rest >= 0 && pos0 >= 0 && (pairing == CC_ROPE_NEIGHBOURS || pairing == CC_ROPE_HALVES), "latent_prepare_append: bad arguments");
+    const int64_t T = q_src->shape[0], cols = (int64_t)n_heads * (dim + rest);
+    CC_REQUIRE(dev, q_col0 >= 0 && q_col0 + cols <= q_src->shape[1], "latent_prepare_append: the queries need %lld columns from column %d on", (long long)cols, q_col0);
+    if (freq) { SEQ_F32(dev, freq, "latent_prepare_append freq"); CC_REQUIRE(dev, 2 * view_len(freq) <= rest, "latent_prepare_append: more rotated pairs than rotated columns"); }
+    LatAppend a{};
+    a.freq = freq ? fptr(freq) : nullptr; a.half = freq ? (int)view_len(freq) : 0; a.step = pairing == CC_ROPE_HALVES ? 1 : 2; a.gap = pairing == CC_ROPE_HALVES ? a.half : 1;
+    a.rest = rest; a.eps = eps; a.mag = mag; a.pos0 = pos0;
+    if (kv_src) {
+        SEQ_ROWS(dev, kv_src, "latent_prepare_append kv"); SEQ_F32(dev, ring, "latent_prepare_append ring");
+        CC_REQUIRE(dev, ring->ndim == 2 && ring->shape[1] > rest && T <= ring->shape[0] && kv_src->shape[0] == T && kv_col0 >= 0 && kv_col0 + ring->shape[1] <= kv_src->shape[1],
+                   "latent_prepare_append: the raw rows need a ring row's columns from column %d on", kv_col0);
+        a.rank = (int)(ring->shape[1] - rest);
+        if (norm_w) { SEQ_F32(dev, norm_w, "latent_prepare_append norm_w"); CC_REQUIRE(dev, view_len(norm_w) == a.rank, "latent_prepare_append: norm_w must have %d elements", a.rank); }
+        a.ring = fptr(ring); a.ckv = fptr(kv_src) + kv_col0; a.nw = norm_w ? fptr(norm_w) : nullptr; a.rs = kv_src->strides[0]; a.ring_rows = (int)ring->shape[0];
+    }
+    cc_buf* o = nullptr;
+    int rc = cc_new_activation(dev, T * cols, CC_F32, false, &o);
+    if (rc) return rc;
+    *out = o;
+    if (T == 0) return CC_OK;
+    latent_prepare_kernel<<<(unsigned)T, 256, 0, dev->stream>>>(fptr(q_src) + q_col0, q_src->strides[0], (float*)o->base, n_heads, dim, a);
+    CC_LAUNCH_CHECK(dev);
+    return CC_OK;
 }
 
 // out[j, h] = [ a[j, h, :dim] | shared[j, col0 : col0 + rest] ]: every head's part followed by the columns all heads share.  One thread per element.

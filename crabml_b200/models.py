@@ -78,3 +78,11 @@ def _load_papunex(path, device, dtype="bfloat16", chunk=0, max_tokens=0, **_):
 
 
 register("Papunex", _load_papunex)
+
+
+def _load_vadodra(path, device, dtype="bfloat16", chunk=0, max_tokens=0, **_):
+    from . import vadodra
+    return vadodra.load(path, device, dtype, chunk, max_tokens)
+
+
+register("Vadodra", _load_vadodra)

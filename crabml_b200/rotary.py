@@ -38,15 +38,23 @@ def wavelength_band_table(dims: int, base: float, factor: float, original: float
     return np.where(wave < original / high, f, np.where(wave > original / low, f / factor, blend)), 1.0
 
 
+def linear_table(dims: int, base: float, factor: float):
+    """linear scaling: every frequency divided by `factor`"""
+    return plain_table(dims, base)[0] / factor, 1.0
+
+
 def table_of(rot: dict):
     """rot: {"dims", "base", optional "scaling"} -> (float32 frequencies [dims / 2], factor on cos and sin).  The scaling's keys say which
-    rule it is: {"factor", "original", "fast", "slow"} is YaRN, {"factor", "original", "low", "high"} the wavelength bands."""
+    rule it is: {"factor"} alone is linear, {"factor", "original", "fast", "slow"} is YaRN, {"factor", "original", "low", "high"} the wavelength
+    bands."""
     dims, base = int(rot["dims"]), float(rot["base"])
     sc = rot.get("scaling")
     if not sc:
         f, mag = plain_table(dims, base)
     elif "low" in sc or "high" in sc:
         f, mag = wavelength_band_table(dims, base, float(sc["factor"]), float(sc["original"]), float(sc["low"]), float(sc["high"]))
+    elif set(sc) == {"factor"}:
+        f, mag = linear_table(dims, base, float(sc["factor"]))
     else:
         f, mag = yarn_table(dims, base, float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"]))
     return f.astype(np.float32), float(mag)

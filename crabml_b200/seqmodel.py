@@ -107,13 +107,13 @@ class Uploader:
         a = self.weights[name]
         return self._mat_from(None, np.asarray(a)) if name in self.bf16_names else self._mat_from(np.asarray(a, np.float32), None)
 
-    def stack(self, names) -> CudaTensor:
-        """the named matrices one under the other (expert-major stacks).  An entry may be (name, cut): cut(array) is stacked instead of the
+    def stack(self, names, axis: int = 0) -> CudaTensor:
+        """the named matrices one under the other (expert-major stacks), with axis = 1 side by side.  An entry may be (name, cut): cut(array) is stacked instead of the
         array; it slices or zero-pads and must not depend on the values (bfloat16 tensors reach it as bit patterns)."""
         names = [n if isinstance(n, tuple) else (n, lambda a: a) for n in names]
         if all(n in self.bf16_names for n, _ in names):
-            return self._mat_from(None, np.concatenate([cut(np.asarray(self.weights[n])) for n, cut in names], 0))
-        return self._mat_from(np.concatenate([cut(self.f32(n)) for n, cut in names], 0), None)
+            return self._mat_from(None, np.concatenate([cut(np.asarray(self.weights[n])) for n, cut in names], axis))
+        return self._mat_from(np.concatenate([cut(self.f32(n)) for n, cut in names], axis), None)
 
     # ---- what mixers of several families upload (csrc/host/mixers.hpp) ------------------------------------------------------------------
     def latent_projections(self, p, heads, dim, kv_rank) -> dict:

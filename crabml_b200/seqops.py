@@ -350,3 +350,52 @@ def feed_forward_act(x, w_up, w_down, act):
     h = C.c_void_p()
     x.device.check(x.device.lib.cc_feed_forward_act(x.device.handle, _v(x), _v(w_up), _v(w_down), int(act), C.byref(h)))
     return _new(x.device, h, list(x.shape()))
+
+
+# ---- a layer whose sublayers stand side by side on one norm; column blocks of its stacked product --------------------------------------------
+def head_gate_cols(x, gate_src, gate_col0, n_heads, act=capi.ACT_SIGMOID):
+    x.device.check(x.device.lib.cc_head_gate_cols(x.device.handle, _v(x), _v(gate_src), int(gate_col0), int(n_heads), int(act)))
+    return x
+
+
+def qk_prepare_append_cols(src, q_col0, k_col0, v_col0, kring, vring, pos0, n_heads, n_kv, dk, dv, qk_norm=capi.QK_NORM_NONE, q_w=None, k_w=None, eps=0.0, freq=None,
+                           pairing=capi.ROPE_NEIGHBOURS, offset=0, mag=1.0):
+    """qk_prepare_append on column blocks of src -> the prepared queries"""
+    h = C.c_void_p()
+    src.device.check(src.device.lib.cc_qk_prepare_append_cols(src.device.handle, _v(src), int(q_col0), int(k_col0), int(v_col0), _v(kring), _v(vring), int(qk_norm), _v(q_w), _v(k_w),
+                                                              float(eps), _v(freq), int(pairing), int(offset), float(mag), int(pos0), n_heads, n_kv, dk, dv, C.byref(h)))
+    return _new(src.device, h, [src.shape()[0], n_heads * dk])
+
+
+def head_project_head_gated(x, w, n_heads, gate_src, gate_col0=0):
+    h = C.c_void_p()
+    x.device.check(x.device.lib.cc_head_project_head_gated(x.device.handle, _v(x), _v(w), int(n_heads), _v(gate_src), int(gate_col0), C.byref(h)))
+    return _new(x.device, h, [x.shape()[0], w.shape()[0]])
+
+
+def latent_query_append_paired(q_src, q_col0, uk_t, n_heads, rest, freq, pairing, mag, pos0, kv_src=None, kv_col0=0, ring=None, norm_w=None, eps=0.0):
+    h = C.c_void_p()
+    q_src.device.check(q_src.device.lib.cc_latent_query_append_paired(q_src.device.handle, _v(q_src), int(q_col0), _v(uk_t), int(n_heads), int(rest), _v(freq), int(pairing), float(mag),
+                                                                      int(pos0), _v(kv_src), int(kv_col0), _v(ring), _v(norm_w), float(eps), C.byref(h)))
+    return _new(q_src.device, h, [q_src.shape()[0], uk_t.shape()[0] + n_heads * rest])
+
+
+def latent_prepare_append(q_src, q_col0, n_heads, dim, rest, freq, pairing, mag, pos0, kv_src=None, kv_col0=0, ring=None, norm_w=None, eps=0.0):
+    """the rotated queries of a pass of many rows; with kv_src also writes the tokens' cache rows"""
+    h = C.c_void_p()
+    q_src.device.check(q_src.device.lib.cc_latent_prepare_append(q_src.device.handle, _v(q_src), int(q_col0), int(n_heads), int(dim), int(rest), _v(freq), int(pairing), float(mag),
+                                                                 int(pos0), _v(kv_src), int(kv_col0), _v(ring), _v(norm_w), float(eps), C.byref(h)))
+    return _new(q_src.device, h, [q_src.shape()[0], n_heads * (dim + rest)])
+
+
+def layer_norm_product(x, norm_w, norm_b, eps, w):
+    h = C.c_void_p()
+    x.device.check(x.device.lib.cc_layer_norm_product(x.device.handle, _v(x), _v(norm_w), _v(norm_b), float(eps), _v(w), C.byref(h)))
+    return _new(x.device, h, [x.shape()[0], w.shape()[0]])
+
+
+def joined_product_accumulate(dst, w, a, src=None, gate_col0=0, up_col0=0, ff=0, act=capi.ACT_SILU, alpha=1.0, limit=0.0, up_shift=0.0):
+    """dst += w [a | gated units of src's columns]"""
+    P = capi.cc_glu_params(int(act), float(alpha), float(limit), float(up_shift))
+    dst.device.check(dst.device.lib.cc_joined_product_accumulate(dst.device.handle, _v(dst), _v(w), _v(a), _v(src), int(gate_col0), int(up_col0), int(ff), C.byref(P)))
+    return dst

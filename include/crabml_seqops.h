@@ -80,6 +80,8 @@ CC_API int cc_scaled_sum(cc_device* dev, const cc_view* dst, const cc_view* a, f
 CC_API int cc_scaled_sum_accumulate(cc_device* dev, const cc_view* dst, const cc_view* a, float sa, const cc_view* b, float sb, const cc_view* c);
 /* x[t, h, :] *= act(g[t, h]): ONE gate number per (row, head) on the head's whole output.  x: [rows, heads * head_size], g: [rows, heads]. */
 CC_API int cc_head_gate(cc_device* dev, const cc_view* x, const cc_view* g, int32_t n_heads, int32_t act);
+/* cc_head_gate with the gate numbers in the columns gate_col0 .. gate_col0 + n_heads of gate_src's rows (a block of a stacked product's result) */
+CC_API int cc_head_gate_cols(cc_device* dev, const cc_view* x, const cc_view* gate_src, int32_t gate_col0, int32_t n_heads, int32_t act);
 /* out = [a | b], row by row: a [rows, ca], b [rows, cb] -> out [rows, ca + cb] (two streams that enter one product side by side) */
 CC_API int cc_concat_cols(cc_device* dev, const cc_view* a, const cc_view* b, cc_buf** out);
 
@@ -221,6 +223,12 @@ enum cc_rope_pairing { CC_ROPE_NEIGHBOURS = 0, CC_ROPE_HALVES = 1 };
 CC_API int cc_qk_prepare_append(cc_device* dev, const cc_view* q, const cc_view* k, const cc_view* v, const cc_view* kring, const cc_view* vring, int32_t qk_norm,
                                 const cc_view* q_w, const cc_view* k_w, float eps, const cc_view* freq, int32_t pairing, int32_t offset, float mag, int64_t pos0,
                                 int32_t n_heads, int32_t n_kv, int32_t dk, int32_t dv);
+/* cc_qk_prepare_append on column blocks of one stacked product's result src [T, >= ...]: raw queries in the columns q_col0 .., keys k_col0 ..,
+ * values v_col0 ..; src stays as it is, the prepared queries come out as [T, n_heads * dk].  v_col0 may be k_col0: the values are then the keys
+ * as projected, before their norm and rotation. */
+CC_API int cc_qk_prepare_append_cols(cc_device* dev, const cc_view* src, int32_t q_col0, int32_t k_col0, int32_t v_col0, const cc_view* kring, const cc_view* vring,
+                                     int32_t qk_norm, const cc_view* q_w, const cc_view* k_w, float eps, const cc_view* freq, int32_t pairing, int32_t offset, float mag,
+                                     int64_t pos0, int32_t n_heads, int32_t n_kv, int32_t dk, int32_t dv, cc_buf** out);
 
 /* ---- latent key/value cache --------------------------------------------------------------------------------------------------- */
 /* A cache row is [c | r]: c, `rank` numbers from which keys and values of all heads derive, and r, a rotated key part that all heads
@@ -242,12 +250,23 @@ CC_API int cc_head_project(cc_device* dev, const cc_view* x, const cc_view* w, i
 /* cc_head_project without carried columns and with a gate on the result: out[t, h] = (W_h x[t, h]) * sigmoid(g[t, h]), g the columns
  * gate_col0 .. gate_col0 + heads * n_out of gate_src's rows (a block of a stacked product's result) */
 CC_API int cc_head_project_gated(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, cc_buf** out);
+/* The same with ONE gate number per head: out[t, h] = (W_h x[t, h]) * sigmoid(g[t, h]), g the columns gate_col0 .. gate_col0 + heads */
+CC_API int cc_head_project_head_gated(cc_device* dev, const cc_view* x, const cc_view* w, int32_t n_heads, const cc_view* gate_src, int32_t gate_col0, cc_buf** out);
 /* What a decoding pass of latent attention does between its projections and the scores, in one kernel: the queries' fold
  * (cc_head_project with carried columns rotated on the way; queries in the columns q_col0 .. of q_src's rows, uk_t: [heads * rank, dim])
  * and the cache rows of the same tokens (cc_latent_ring_append; raw rows in the columns kv_col0 .. of kv_src).  kv_src NULL: nothing is
  * appended (a layer that reads another layer's cache; ring and norm_w are ignored).  out: [T, heads * (rank + rest)]. */
 CC_API int cc_latent_query_append(cc_device* dev, const cc_view* q_src, int32_t q_col0, const cc_view* uk_t, int32_t n_heads, int32_t rest, const cc_view* freq, float mag,
                                   int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps, cc_buf** out);
+
+/* cc_latent_query_append with the pairing of the rotated columns as a parameter (cc_rope_pairing; the plain one pairs neighbours) */
+CC_API int cc_latent_query_append_paired(cc_device* dev, const cc_view* q_src, int32_t q_col0, const cc_view* uk_t, int32_t n_heads, int32_t rest, const cc_view* freq,
+                                         int32_t pairing, float mag, int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps,
+                                         cc_buf** out);
+/* What a pass of many rows does there, where queries are not folded: they leave their columns as out [T, heads * (dim + rest)], the last `rest`
+ * columns of every head rotated, and the same tokens' cache rows are written (kv_src NULL: none; ring and norm_w are then ignored). */
+CC_API int cc_latent_prepare_append(cc_device* dev, const cc_view* q_src, int32_t q_col0, int32_t n_heads, int32_t dim, int32_t rest, const cc_view* freq, int32_t pairing,
+                                    float mag, int64_t pos0, const cc_view* kv_src, int32_t kv_col0, const cc_view* ring, const cc_view* norm_w, float eps, cc_buf** out);
 
 /* out[j, h] = [ a[j, h] | shared[j, col0 : col0 + rest] ]: a: [rows, heads * dim]; shared: [>= rows, cols] (its first `rows` rows are used);
  * out: [rows, heads * (dim + rest)].  Builds per-head keys out of their own part and a part all heads share (a latent cache's rotated columns). */
@@ -296,6 +315,16 @@ CC_API int cc_moe_experts_act(cc_device* dev, const cc_view* x, const cc_view* i
                               int32_t ff, int32_t act, cc_buf** out);
 /* the same unit for every token: out = W_down act(W_up x) ; w_up: [ff, D], w_down: [D, ff], both F32 or both BF16 */
 CC_API int cc_feed_forward_act(cc_device* dev, const cc_view* x, const cc_view* w_up, const cc_view* w_down, int32_t act, cc_buf** out);
+
+/* ---- the products of a layer whose sublayers stand side by side on one norm ---------------------------------------------------- */
+/* out = W LN(x): cc_layer_norm (norm_b may be NULL), then cc_matmul_vec; the normed rows are only the product's operand.  x: [T, k]; w: [m, k],
+ * F32 or BF16.  out: [T, m]. */
+CC_API int cc_layer_norm_product(cc_device* dev, const cc_view* x, const cc_view* norm_w, const cc_view* norm_b, float eps, const cc_view* w, cc_buf** out);
+/* dst += W [a | unit(g, u)], the output projections of two sublayers side by side as ONE product whose sum joins the residual stream: w [m, ca + ff]
+ * is [W_a | W_b], a [T, ca] the one sublayer's result, g and u the columns gate_col0 .. and up_col0 .. (ff each) of src's rows, unit the gated
+ * unit of cc_glu_params.  ff = 0: dst += W a (src and glu may be NULL).  dst: [T, m]. */
+CC_API int cc_joined_product_accumulate(cc_device* dev, const cc_view* dst, const cc_view* w, const cc_view* a, const cc_view* src, int32_t gate_col0, int32_t up_col0,
+                                        int32_t ff, const cc_glu_params* glu);
 
 #ifdef __cplusplus
 }
