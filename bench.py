@@ -53,6 +53,10 @@ WORKLOADS = {
     "papunex-w1024": ("PAPUNEX", "BF16", "BF16"),
     "papunex-w2048": ("PAPUNEX", "BF16", "BF16"),
     "papunex-w4096": ("PAPUNEX", "BF16", "BF16"),
+    # the Vadodra family at the same layer sizes, beside the Lifesun and Papunex stacks of equal width and depth; see run_vadodra
+    "vadodra-w1024": ("VADODRA", "BF16", "BF16"),
+    "vadodra-w2048": ("VADODRA", "BF16", "BF16"),
+    "vadodra-w4096": ("VADODRA", "BF16", "BF16"),
 }
 # dram bytes per megakernel launch from the committed ncu --set full capture (profiles/); None until captured
 TRAFFIC = {("llama2-7b-q8_0", 1): 7040893000 + 49879296}     # profiles/r02p_mega_ring_q8_0_ncu_raw.csv (mega_ring_kernel: dram__bytes_read.sum + dram__bytes_write.sum)
@@ -931,6 +935,136 @@ def run_papunex(args, rank, world, local_rank):
     print(json.dumps(line))
 
 
+def vadodra_bench_config(width: int, vocab: int = 32000):
+    """four layers, each with a dense feed-forward of 3 x width, as in the Lifesun stack: window attention (1024 positions, 128-wide heads, 4 query
+    heads per key head, half of every head rotated) and causal latent attention (128 + 64 wide query heads over a latent of 512), alternating; the
+    second latent layer reads the first one's cache"""
+    H = width // 128
+    win = {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+           "rot": {"dims": 64, "base": 200000.0, "scaling": {"factor": 4.0}}}
+    lat = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": {"dims": 64, "base": 10000.0}}
+    mlp = {"kind": "dense", "ff": 3 * width, "limit": 7.0}
+    layers = [{"type": "attention", "mixer": win, "mlp": mlp}, {"type": "latent_attention", "mixer": lat, "mlp": mlp}, {"type": "attention", "mixer": win, "mlp": mlp},
+              {"type": "latent_attention", "mixer": dict(lat, kv_from=1), "mlp": mlp}]
+    return {"architecture": "Vadodra", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def time_vadodra_kernels(dev, width, T):
+    """The steps of a Vadodra layer that no other family has, alone at the bench's sizes, beside the steps the other families would take for the
+    same function: for a pass of T rows (floating-point operations per second of the products, bytes per second of the rest) and for one
+    decoded row (weight bytes per second)."""
+    from crabml_b200 import CudaTensor, capi, seqops
+    from crabml_b200.safetensors import f32_to_bf16
+    rng = np.random.default_rng(SEED)
+
+    def rand(*shape):
+        return CudaTensor.new(rng.standard_normal(shape).astype(np.float32), list(shape), dev)
+
+    def mat(a):
+        return CudaTensor.from_cpu(np.ascontiguousarray(f32_to_bf16(a).reshape(a.shape)), list(a.shape), capi.BF16, dev)
+
+    def draw(*shape):
+        return (rng.standard_normal(shape) / np.sqrt(shape[-1])).astype(np.float32)
+    out = {}
+    flush = rand(48 * 1024 * 1024)                                     # 192 MB: read and written between timed calls, so that no call finds its weights in L2
+
+    def timed(name, f, reps=5, **what):
+        f()
+        ms = 0.0
+        for _ in range(reps):
+            seqops.activate_inplace(flush, capi.ACT_NONE)
+            dev.synchronize(); dev.timer_begin()
+            f()
+            ms += dev.timer_end()
+        out[name] = dict(what, ms=ms / reps)
+        for k in ("flop", "bytes"):
+            if k in what:
+                out[name][k + "_per_s"] = what[k] / (ms / reps * 1e-3)
+    D, H = width, width // 128
+    G, ff = max(1, H // 4), 3 * width
+    qk = H * 128 + G * 128
+    m_in, k_out = qk + 2 * ff, H * 128 + ff
+    o, down = draw(D, H * 128), draw(D, ff)
+    w_in, w_o, w_down, w_out = mat(draw(m_in, D)), mat(o), mat(down), mat(np.concatenate([o, down], 1))
+    norm, qn = rand(D), rand(128)
+    freq = CudaTensor.new(np.power(2e5, -np.arange(32) / 32.0).astype(np.float32) / 4, [32], dev)
+    kr, vr = rand(1024 + T, G * 128), rand(1024 + T, G * 128)
+    uk_t, ring, gates = rand(H * 512, 128), rand(4096, 576), rand(T, H)
+    for rows, tag in ((T, "prompt"), (1, "decode")):
+        x, a, src = rand(rows, D), rand(rows, H * 128), rand(rows, m_in)
+        unit = dict(act=capi.ACT_SWISH, alpha=1.702, limit=7.0, up_shift=1.0)
+        what_in, what_out = ({"flop": 2 * rows * D * m_in}, {"flop": 2 * rows * D * k_out}) if rows > 1 else ({"bytes": 2 * D * m_in}, {"bytes": 2 * D * k_out})
+        timed(f"{tag}: norm and input product", lambda: seqops.layer_norm_product(x, norm, None, 1e-5, w_in), rows=rows, **what_in)
+        timed(f"{tag}: norm, then the product (closest model)", lambda: w_in.matmul_vec(seqops.layer_norm(x, norm, None, 1e-5)), rows=rows, **what_in)
+        timed(f"{tag}: joined output product with gated units and residual", lambda: seqops.joined_product_accumulate(x, w_out, a, src, qk, qk + ff, ff, **unit), rows=rows, **what_out)
+        gu = rand(rows, 2 * ff)
+        timed(f"{tag}: two output products, gated units, residual sum (closest model)",
+              lambda: seqops.scaled_sum_accumulate(x, w_o.matmul_vec(a), 1.0, w_down.matmul_vec(seqops.glu_halves(gu, None, capi.ACT_GELU_TANH)), 1.0), rows=rows, **what_out)
+        q, k = rand(rows, H * 128), rand(rows, G * 128)
+        prep = {"rows": rows, "bytes": rows * (2 * H + 3 * G) * 128 * 4}
+        args = dict(qk_norm=capi.QK_NORM_HEAD, q_w=qn, k_w=qn, eps=1e-5, freq=freq, pairing=capi.ROPE_NEIGHBOURS)
+        timed(f"{tag}: queries and keys from columns to rings", lambda: seqops.qk_prepare_append_cols(src, 0, H * 128, H * 128, kr, vr, 100, H, G, 128, 128, **args), **prep)
+        timed(f"{tag}: queries and keys from tensors to rings (closest model)", lambda: seqops.qk_prepare_append(q, k, k, kr, vr, 100, H, G, 128, 128, **args), **prep)
+        ls = rand(rows, H * 192 + H + 576)
+        lat = {"rows": rows, "bytes": rows * (2 * H * 192 + 2 * 576) * 4}
+        if rows > 1:
+            timed(f"{tag}: latent queries and cache rows from columns", lambda: seqops.latent_prepare_append(ls, 0, H, 128, 64, freq, capi.ROPE_HALVES, 1.0, 100, ls, H * 193, ring), **lat)
+            timed(f"{tag}: cut, rotation, cache rows (closest model)", lambda: _latent_parts(seqops, ls, H, ring, freq), **lat)
+            timed(f"{tag}: gate per head from columns", lambda: seqops.head_gate_cols(a, ls, H * 192, H), rows=rows, bytes=2 * rows * H * 128 * 4)
+            timed(f"{tag}: gate per element (closest model)", lambda: seqops.gated_sum(a, a, g1=q, accumulate=False), rows=rows, bytes=3 * rows * H * 128 * 4)
+        else:
+            fold = {"rows": 1, "bytes": H * 512 * 128 * 4}
+            timed(f"{tag}: query fold and cache row, halves", lambda: seqops.latent_query_append_paired(ls, 0, uk_t, H, 64, freq, capi.ROPE_HALVES, 1.0, 100, ls, H * 193, ring), **fold)
+            timed(f"{tag}: query fold and cache row (closest model)", lambda: seqops.latent_query_append(ls, 0, uk_t, H, 64, freq, 1.0, 100, ls, H * 193, ring), **fold)
+            ol, uv = rand(1, H * 512), rand(H * 128, 512)
+            timed(f"{tag}: value up-projection, gate per head", lambda: seqops.head_project_head_gated(ol, uv, H, ls, H * 192), **fold)
+            timed(f"{tag}: value up-projection, gate per element (closest model)", lambda: seqops.head_project_gated(ol, uv, H, q, 0), **fold)
+    return out
+
+
+def _latent_parts(seqops, src, H, ring, freq):
+    q, _, kv = seqops.split_cols(src, [H * 192, H, 576])
+    seqops.latent_ring_append(ring, kv, None, 1e-5, 512, freq, 1.0, 100)
+    return seqops.rope_pairs(q, H, 192, 128, freq, 1.0, 100)
+
+
+def run_vadodra(args, rank, world, local_rank):
+    """Prefill and decode throughput of the Vadodra family at real layer sizes, beside the closest existing models -- the Lifesun stack (one layer
+    norm feeding parallel sublayers, window attention) and the Papunex stack (latent attention with a shared cache) of the same width, depth and
+    active feed-forward width -- through the same step function and slots; then the steps of a layer that no other family has."""
+    from crabml_b200 import CudaTensorDevice, lifesun, papunex, vadodra
+    if rank != 0:
+        return
+    width = int(args.workload.split("-w")[1])
+    Tp, K, W = args.prefill_tokens, args.steps, args.warmup
+    rng = np.random.default_rng(SEED)
+    prompt = [int(v) for v in rng.integers(0, 32000, Tp)]
+    sampler = ClockSampler(local_rank); sampler.start()
+    out = {}
+    for name, mod, cls, raw in (("vadodra", vadodra, "VadodraModel", vadodra_bench_config(width)), ("lifesun", lifesun, "LifesunModel", lifesun_bench_config(width)),
+                                ("papunex", papunex, "PapunexModel", papunex_bench_config(width))):
+        conf = mod.parse_config(raw)
+        dev = CudaTensorDevice(local_rank, lazy=0)
+        weights = mod.random_weights(conf, SEED)
+        model = getattr(mod, cls)(dev, conf, weights, "bfloat16", chunk=args.zatorax_chunk, max_seq=Tp + K + W + 8)
+        params = sum(int(np.prod(np.shape(a))) for a in weights.values())
+        del weights
+        out[name] = measure_seq_model(dev, model, prompt, K, W, params)
+        model.close()
+        if name == "vadodra":
+            out["layer_steps"] = time_vadodra_kernels(dev, width, args.zatorax_chunk)
+        dev.close()
+    clocks = sampler.stop()
+    z = out["vadodra"]
+    line = {"metric": "decode_tokens_per_s", "value": z["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": z["decode_ms_per_token"],
+            "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 matrices and product inputs, f32 everything else", "data": "synthetic",
+            "config": {"workload": args.workload, "model": vadodra_bench_config(width), "prefill_tokens": Tp, "chunk": args.zatorax_chunk,
+                       "closest_models": {"lifesun": lifesun_bench_config(width), "papunex": papunex_bench_config(width)}},
+            "e2e": {"value": 1e3 / z["decode_wall_ms_per_token"], "unit": "tok/s", "h2d_bytes_per_step": 8, "d2h_bytes_per_step": 32000 * 4},
+            "gpu_launches": int(z["decode_launches_per_token"] * K), "detail": out, "clocks": clocks}
+    print(json.dumps(line))
+
+
 def run_zatorax(args, rank, world, local_rank):
     """Prefill and decode throughput of the Zatorax family at real layer sizes, beside the closest existing model -- a llama stack of the
     same width, depth, head layout and ACTIVE feed-forward width (Q8_0 weights, its serving format) -- through each family's runner.
@@ -1008,7 +1142,7 @@ def main():
     ap.add_argument("--no-also", action="store_true", help="skip the second (Q4_0) measurement of the default run")
     ap.add_argument("--multi", default="sharded", choices=["sharded", "replicas"], help="N > 1: shard one token stream (strong scaling, default) or run N independent replicas")
     ap.add_argument("--comm", default="p2p", choices=["p2p", "nccl"], help="exchange transport of the sharded path: one-shot NVLink peer stores (default) or the NCCL baseline")
-    ap.add_argument("--zatorax-chunk", type=int, default=512, help="zatorax / meresun / vuzinex / lifesun / papunex workloads: longest run of prompt tokens one pass takes")
+    ap.add_argument("--zatorax-chunk", type=int, default=512, help="zatorax / meresun / vuzinex / lifesun / papunex / vadodra workloads: longest run of prompt tokens one pass takes")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -1025,6 +1159,8 @@ def main():
         run_lifesun(args, rank, world, local_rank)
     elif args.workload.startswith("papunex-"):
         run_papunex(args, rank, world, local_rank)
+    elif args.workload.startswith("vadodra-"):
+        run_vadodra(args, rank, world, local_rank)
     elif args.workload.endswith("-prefill"):
         run_prefill(args, rank, world, local_rank)
     else:
