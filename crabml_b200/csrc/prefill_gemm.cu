@@ -392,16 +392,34 @@ int cc_prefill_bf16_operand(cc_device* dev, int64_t b, int64_t k, void** out) {
     *out = s->x;
     return rc;
 }
+// The output tile of a CTA: large tiles read fewer operand bytes per multiplication, small ones put more SMs to work.  Estimated time of a tile in
+// SM cycles: per 64-deep step the slowest of the tensor core (4096 multiply-adds per cycle), the operand bytes at about 40 per cycle and a floor
+// for the step's own latency; once per tile its start and its stores.  The whole product takes as many rounds of tiles as the SMs need.
+static void pg_pick_tile(cc_device* dev, int64_t m, int64_t b, int64_t k, int* block_n, int* mt) {
+    double best = 0.0;
+    for (int n = 256; n >= 64; n /= 2)
+        for (int t = 2; t >= 1; t--) {
+            if (n > 64 && b <= n / 2) continue;                  // more than half of every tile would be padding
+            const int64_t tiles = ((m + PG_BLOCK_M * t - 1) / (PG_BLOCK_M * t)) * ((b + n - 1) / n);
+            const int64_t rounds = (tiles + dev->sm_count - 1) / dev->sm_count;
+            const double mma = t * PG_BLOCK_M * (double)n * PG_BLOCK_K / 4096.0, load = (t * PG_BLOCK_M + n) * PG_BLOCK_K * 2 / 40.0;
+            double step = mma > load ? mma : load;
+            if (step < 260.0) step = 260.0;
+            const double cost = rounds * (step * (k / PG_BLOCK_K) + 3000.0 + t * n * 8.0);
+            if (best == 0.0 || cost < best) { best = cost; *block_n = n; *mt = t; }
+        }
+}
 // the product over the operand in that scratch; accumulate != 0: out += it
 int cc_launch_prefill_bf16_operand(cc_device* dev, const cc_buf* w, float* out, int64_t m, int64_t k, int64_t b, int accumulate) {
     PgScratch* s = pg_scratch(dev);
-    const int block_n = b >= 192 ? 256 : b >= 96 ? 128 : 64;
+    int block_n = 64, mt = 1;
+    pg_pick_tile(dev, m, b, k, &block_n, &mt);
     CUtensorMap tw, tx;
     int rc = pg_make_tmap(dev, &tw, w->plane[0], m, k, PG_BLOCK_M, true);
     if (rc) return rc;
     rc = pg_make_tmap(dev, &tx, s->x, b, k, block_n, true);
     if (rc) return rc;
-    const bool mt2 = m >= 512;
+    const bool mt2 = mt == 2;
     if (block_n == 256) return mt2 ? pg_launch<256, 2, 1>(dev, tw, tx, out, m, b, k, accumulate) : pg_launch<256, 1, 1>(dev, tw, tx, out, m, b, k, accumulate);
     if (block_n == 128) return mt2 ? pg_launch<128, 2, 1>(dev, tw, tx, out, m, b, k, accumulate) : pg_launch<128, 1, 1>(dev, tw, tx, out, m, b, k, accumulate);
     return mt2 ? pg_launch<64, 2, 1>(dev, tw, tx, out, m, b, k, accumulate) : pg_launch<64, 1, 1>(dev, tw, tx, out, m, b, k, accumulate);

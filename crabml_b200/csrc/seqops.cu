@@ -6,6 +6,7 @@
 // contents, never on how many tokens the call carries or where the token sits in the call.  Sums run in a fixed order per output
 // (a warp's lane-strided partial sums and the xor butterfly, or one thread's sequential loop), so prefill, chunked prefill and
 // token-by-token decoding give the same bits for the recurrent layers and the same bits per (query, key set) for attention.
+#include <cooperative_groups.h>
 #include <cuda_bf16.h>
 
 #include "../../include/crabml_seqops.h"
@@ -726,8 +727,8 @@ extern "C" CC_API int cc_kv_ring_append(cc_device* dev, const cc_view* kring, co
 //   3. wa_values_kernel : out[row][d] = sum_c S[row][c] v[lo_i + c][d], a 64 x 64 tile product over the keys of the tile's band
 // A row is one (query, head); a tile's 64 rows are the R = n_heads / n_kv heads of one key/value head for 64 / R consecutive queries.
 // Every dot product runs over its index in ascending order inside ONE thread, the softmax sums depend on the row alone, and the value sum
-// has one order per kernel (ascending keys in the tile kernel, masked keys adding an exact 0; four ascending quarters in the row kernel that
-// serves calls of few rows): a query's result does not depend on where the call starts or what else it carries, and differs between a
+// has one order per kernel (ascending keys in the tile kernel, masked keys adding an exact 0; ascending slices in the kernel that serves calls
+// of few rows): a query's result does not depend on where the call starts or what else it carries, and differs between a
 // prompt pass and a decoded token only by the rounding of that last sum.
 #define WA_TILE 64
 #define WA_K 16
@@ -773,18 +774,23 @@ __global__ void __launch_bounds__(WA_THREADS) wa_scores_kernel(const float* __re
     for (int a = 0; a < 4; a++)
 #pragma unroll
         for (int b = 0; b < 4; b++) acc[a][b] = 0.0f;
-    // the next 16 coordinates of queries and keys are fetched into registers while the current ones are multiplied
+    // the next 16 coordinates of queries and keys are fetched into registers while the current ones are multiplied; a thread's rows stay the same
     float pq[4], pk[4];
+    const float *qp[4], *kp[4];
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        const int r = (threadIdx.x + e * WA_THREADS) >> 4;
+        const int tq = r / g.R, hr = r - tq * g.R;
+        const int64_t j = j0 + r;
+        qp[e] = tq < tq_n ? q + ((int64_t)(t0 + tq) * g.H + kvh * g.R + hr) * g.dk : nullptr;
+        kp[e] = j <= i_last ? kring + (j % g.ring) * g.krs + kvh * g.dk : nullptr;
+    }
     auto fetch = [&](int d0) {
+        const int d = d0 + (threadIdx.x & 15);
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-            const int idx = threadIdx.x + e * WA_THREADS;
-            const int r = idx >> 4, dd = idx & 15;
-            const int tq = r / g.R, hr = r - tq * g.R;
-            const bool din = d0 + dd < g.dk;
-            pq[e] = (din && tq < tq_n) ? q[((int64_t)(t0 + tq) * g.H + kvh * g.R + hr) * g.dk + d0 + dd] : 0.0f;
-            const int64_t j = j0 + r;
-            pk[e] = (din && j <= i_last) ? kring[(j % g.ring) * g.krs + kvh * g.dk + d0 + dd] : 0.0f;
+            pq[e] = (d < g.dk && qp[e]) ? qp[e][d] : 0.0f;
+            pk[e] = (d < g.dk && kp[e]) ? kp[e][d] : 0.0f;
         }
     };
     fetch(0);
@@ -828,28 +834,46 @@ __global__ void __launch_bounds__(WA_THREADS) wa_scores_kernel(const float* __re
         }
     }
 }
-// few rows (decoding): grid (ceil(keys / 8), T, G), 256 threads.  The CTA stages the R queries of (token, key/value head); a warp owns one
-// visible key and takes its dot product with each of them: lane-strided partial sums, then the butterfly.  The key row is read once for all
-// R heads, and the keys spread over the whole device however few rows the call has.
+// few rows (decoding): grid (ceil(keys / 16), T, G * head blocks), 256 threads.  The CTA stages up to WS_HEADS queries of (token, key/value head); a
+// warp owns two visible keys and takes their dot products with each of them: lane-strided partial sums, then the butterfly.  A key row is
+// read into registers once for the block's heads (rows longer than WS_KEEP * 32: as far as they fit), and the keys spread over the whole device
+// however few rows the call has.
+#define WS_HEADS 8
+#define WS_KEEP 20
 __global__ void __launch_bounds__(256) wa_scores_row_kernel(const float* __restrict__ q, const float* __restrict__ kring, float* __restrict__ S, WaGeom g, float scale,
                                                             const float* __restrict__ r1, const float* __restrict__ r2) {
-    extern __shared__ float wsr_sm[];             // [R][dk]
-    const int t = blockIdx.y, kvh = blockIdx.z;
+    extern __shared__ float wsr_sm[];             // [heads of the block][dk]
+    const int hblocks = (g.R + WS_HEADS - 1) / WS_HEADS;
+    const int t = blockIdx.y, kvh = blockIdx.z / hblocks, h0 = (blockIdx.z % hblocks) * WS_HEADS, nh = min(WS_HEADS, g.R - h0);
     const int64_t i = g.pos0 + t, lo = wa_lo(g, i);
-    for (int e = threadIdx.x; e < g.R * g.dk; e += 256) wsr_sm[e] = q[((int64_t)t * g.H + kvh * g.R) * g.dk + e];
-    __syncthreads();
     const int lane = threadIdx.x & 31;
-    const int64_t j = lo + (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (j > i) return;
-    const float* kr = kring + (j % g.ring) * g.krs + kvh * g.dk;
-    for (int hr = 0; hr < g.R; hr++) {
+    if (lo + (int64_t)blockIdx.x * 16 > i) return;            // the whole CTA lies behind the last visible key
+    const int64_t ja = lo + (int64_t)blockIdx.x * 16 + (threadIdx.x >> 5), jb = ja + 8;
+    const float* ka = kring + ((ja < i ? ja : i) % g.ring) * g.krs + kvh * g.dk;
+    const float* kb = kring + ((jb < i ? jb : i) % g.ring) * g.krs + kvh * g.dk;
+    float xa[WS_KEEP], xb[WS_KEEP];
+#pragma unroll
+    for (int e = 0; e < WS_KEEP; e++) {
+        const int d = lane + e * 32;
+        xa[e] = d < g.dk ? ka[d] : 0.0f;
+        xb[e] = d < g.dk ? kb[d] : 0.0f;
+    }
+    for (int e = threadIdx.x; e < nh * g.dk; e += 256) wsr_sm[e] = q[((int64_t)t * g.H + kvh * g.R + h0) * g.dk + e];
+    __syncthreads();
+    for (int hr = 0; hr < nh; hr++) {
         const float* qh = wsr_sm + hr * g.dk;
-        float acc = 0.0f;
-        for (int d = lane; d < g.dk; d += 32) acc = fmaf(qh[d], kr[d], acc);
-        acc = warp_sum(acc);
-        if (lane == 0) {
-            const int h = kvh * g.R + hr;
-            float sc = acc * scale;
+        float sa = 0.0f, sb = 0.0f;
+#pragma unroll
+        for (int e = 0; e < WS_KEEP; e++) {
+            const int d = lane + e * 32;
+            if (d < g.dk) { sa = fmaf(qh[d], xa[e], sa); sb = fmaf(qh[d], xb[e], sb); }
+        }
+        for (int d = lane + WS_KEEP * 32; d < g.dk; d += 32) { sa = fmaf(qh[d], ka[d], sa); sb = fmaf(qh[d], kb[d], sb); }
+        sa = warp_sum(sa); sb = warp_sum(sb);
+        const int64_t j = lane ? jb : ja;                     // lane 0 finishes the first key, lane 1 the second
+        if (lane < 2 && j <= i) {
+            const int h = kvh * g.R + h0 + hr;
+            float sc = (lane ? sb : sa) * scale;
             if (g.softcap > 0.0f) sc = g.softcap * tanhf(sc / g.softcap);
             if (r1) sc -= r1[h] * log1pf(r2[h] * (float)(i - j));
             S[((int64_t)t * g.H + h) * g.cap + (j - lo)] = sc;
@@ -877,122 +901,97 @@ __global__ void wa_softmax_kernel(float* __restrict__ S, WaGeom g, const float* 
     const float inv = 1.0f / sum;
     for (int c = lane; c < n; c += 32) Sr[c] *= inv;
 }
-// few rows (decoding): grid (rows, ceil(dv / 32)); a CTA owns 32 output columns of one row = (query, head).  The row's probabilities go to
-// shared memory; the visible keys are cut into four contiguous quarters, warp w adds quarter w in ascending order for its lane's column,
-// and the quarters are added as (p0 + p1) + (p2 + p3).  The order depends on the row alone (its number of visible keys), not on T.
-// S holds the raw scores: every CTA of a row redoes the row's softmax in shared memory (warp 0, the sums in wa_softmax_kernel's order, so the
-// weights are the same bits), which saves a launch per layer in decoding.
-__global__ void __launch_bounds__(128) wa_values_row_kernel(const float* __restrict__ S, const float* __restrict__ vring, float* __restrict__ out, WaGeom g,
-                                                            const float* __restrict__ sink) {
-    extern __shared__ float wr_sm[];
-    __shared__ float part[4][32];
-    const int64_t row = blockIdx.x;
-    const int t = (int)(row / g.H), h = (int)(row % g.H), kvh = h / g.R;
+// few rows (decoding): grid (T * G * head blocks, ceil(dv / 32), WV_SPLIT) in clusters of WV_SPLIT CTAs along z.  A cluster owns 32 value columns of
+// RB query heads of one (token, key/value head), each of its CTAs one contiguous slice of the visible keys: raw scores of the slice -> its
+// largest score, weights relative to it and their sum (a warp per head), then the slice's value rows, each read once for the RB heads
+// (warp w takes the w-th stretch of the slice in ascending order, the warps' sums are added in ascending order).  The slices meet through the
+// cluster's shared memory: rank r finishes the heads r, r + WV_SPLIT, ..., adding the slices in ascending order, each scaled from its own largest
+// score to the common one, the sink with them.  The order depends on the row alone (its number of visible keys), not on T.
+#define WV_SPLIT 8
+#define WV_THREADS 256
+#define WV_WARPS (WV_THREADS / 32)
+template <int RB>
+__global__ void __cluster_dims__(1, 1, WV_SPLIT) __launch_bounds__(WV_THREADS) wa_values_slices_kernel(const float* __restrict__ S, const float* __restrict__ vring, float* __restrict__ out,
+                                                                                                       WaGeom g, const float* __restrict__ sink, int slice_cap) {
+    extern __shared__ float wv_sm[];
+    float* pr = wv_sm;                                        // [RB][slice_cap]
+    float* part = wv_sm + (size_t)RB * slice_cap;             // [WV_WARPS][RB][32]
+    __shared__ float top[RB], sum[RB], acc_sm[RB * 32];       // what the cluster reads: the slice's largest score, sum of weights, weighted values
+    cooperative_groups::cluster_group cluster = cooperative_groups::this_cluster();
+    const int hblocks = (g.R + RB - 1) / RB;
+    const int hb = blockIdx.x % hblocks, tk = blockIdx.x / hblocks;
+    const int t = tk / g.G, kvh = tk % g.G, h0 = hb * RB, nh = min(RB, g.R - h0);
     const int64_t i = g.pos0 + t, lo = wa_lo(g, i);
-    const int n = (int)(i - lo + 1);
+    const int n = (int)(i - lo + 1), per_slice = (n + WV_SPLIT - 1) / WV_SPLIT;
+    const int s0 = min(n, (int)blockIdx.z * per_slice), m = min(n, s0 + per_slice) - s0;      // this CTA's keys: s0 .. s0 + m of the visible ones
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
-    for (int c = threadIdx.x; c < n; c += 128) wr_sm[c] = S[row * g.cap + c];
-    __syncthreads();
-    if (w == 0) {
+    for (int hr = w; hr < RB; hr += WV_WARPS) {
+        const float* Sr = S + ((int64_t)t * g.H + kvh * g.R + h0 + hr) * g.cap + s0;
+        float* p = pr + (size_t)hr * slice_cap;
+        const bool on = hr < nh;
         float mx = -INFINITY;
-        for (int c = lane; c < n; c += 32) mx = fmaxf(mx, wr_sm[c]);
+        for (int c = lane; c < m; c += 32) { const float v = on ? Sr[c] : 0.0f; p[c] = v; mx = fmaxf(mx, v); }
         mx = warp_max(mx);
-        const float sk = sink ? sink[h] : -INFINITY;
-        mx = fmaxf(mx, sk);
-        float sum = 0.0f;
-        for (int c = lane; c < n; c += 32) { const float e = expf(wr_sm[c] - mx); wr_sm[c] = e; sum += e; }
-        sum = warp_sum(sum);
-        if (sink) sum += expf(sk - mx);
-        const float inv = 1.0f / sum;
-        for (int c = lane; c < n; c += 32) wr_sm[c] *= inv;
+        float tot = 0.0f;
+        for (int c = lane; c < m; c += 32) { const float e = expf(p[c] - mx); p[c] = e; tot += e; }
+        tot = warp_sum(tot);
+        if (lane == 0) { top[hr] = mx; sum[hr] = tot; }
     }
     __syncthreads();
     const int d = blockIdx.y * 32 + lane;
-    const int per = (n + 3) >> 2;
-    const int c_begin = min(n, w * per), c_end = min(n, c_begin + per);
-    const int r0 = (int)(lo % g.ring);
-    const int64_t rs = g.vrs;
-    float acc = 0.0f;
-    if (d < g.dv) {
-        const float* vb = vring + (int64_t)kvh * g.vhs + d;
-        int r = r0 + c_begin;
-        if (r >= g.ring) r -= g.ring;
-#pragma unroll 8
-        for (int c = c_begin; c < c_end; c++) {
-            acc = fmaf(wr_sm[c], vb[r * rs], acc);
-            if (++r == g.ring) r = 0;
-        }
-    }
-    part[w][lane] = acc;
-    __syncthreads();
-    if (w == 0 && d < g.dv) out[row * g.dv + d] = (part[0][lane] + part[1][lane]) + (part[2][lane] + part[3][lane]);
-}
-// few rows, R > 1 query heads per key/value head: grid (T * G, ceil(dv / 32)), 512 threads.  A CTA owns 32 value columns of ALL R heads of
-// one (token, key/value head), so every value row is read once for the group instead of once per head.  Each head's softmax is redone
-// in shared memory by one warp (wa_softmax_kernel's order); the visible keys are cut into 16 contiguous segments, warp w adds segment w in
-// ascending order into R accumulators per lane, and the segments are added in ascending order.  The order depends on the row alone.
-template <int R>
-__global__ void __launch_bounds__(512) wa_values_group_kernel(const float* __restrict__ S, const float* __restrict__ vring, float* __restrict__ out, WaGeom g,
-                                                              const float* __restrict__ sink) {
-    extern __shared__ float wg_sm[];
-    const int t = blockIdx.x / g.G, kvh = blockIdx.x % g.G;
-    const int64_t i = g.pos0 + t, lo = wa_lo(g, i);
-    const int n = (int)(i - lo + 1);
-    float* pr = wg_sm;                            // [R][n]
-    float* part = wg_sm + (size_t)R * n;          // [16][R][32]
-    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
-    for (int hr = w; hr < R; hr += 16) {
-        const int h = kvh * R + hr;
-        const float* Sr = S + ((int64_t)t * g.H + h) * g.cap;
-        float* p = pr + (size_t)hr * n;
-        float mx = -INFINITY;
-        for (int c = lane; c < n; c += 32) { const float v = Sr[c]; p[c] = v; mx = fmaxf(mx, v); }
-        mx = warp_max(mx);
-        const float sk = sink ? sink[h] : -INFINITY;
-        mx = fmaxf(mx, sk);
-        float sum = 0.0f;
-        for (int c = lane; c < n; c += 32) { const float e = expf(p[c] - mx); p[c] = e; sum += e; }
-        sum = warp_sum(sum);
-        if (sink) sum += expf(sk - mx);
-        const float inv = 1.0f / sum;
-        for (int c = lane; c < n; c += 32) p[c] *= inv;
-    }
-    __syncthreads();
-    const int d = blockIdx.y * 32 + lane;
-    const int per = (n + 15) >> 4;
-    const int c_begin = min(n, w * per), c_end = min(n, c_begin + per);
-    float acc[R];
+    const int per = (m + WV_WARPS - 1) / WV_WARPS;
+    const int c_begin = min(m, w * per), c_end = min(m, c_begin + per);
+    float acc[RB];
 #pragma unroll
-    for (int hr = 0; hr < R; hr++) acc[hr] = 0.0f;
+    for (int hr = 0; hr < RB; hr++) acc[hr] = 0.0f;
     if (d < g.dv) {
         const float* vb = vring + (int64_t)kvh * g.vhs + d;
         const int64_t rs = g.vrs;
-        int r = (int)(lo % g.ring) + c_begin;
-        if (r >= g.ring) r -= g.ring;
-#pragma unroll 4
+        int r = (int)((lo + s0 + c_begin) % g.ring);
+#pragma unroll 8
         for (int c = c_begin; c < c_end; c++) {
             const float v = vb[r * rs];
 #pragma unroll
-            for (int hr = 0; hr < R; hr++) acc[hr] = fmaf(pr[(size_t)hr * n + c], v, acc[hr]);
+            for (int hr = 0; hr < RB; hr++) acc[hr] = fmaf(pr[(size_t)hr * slice_cap + c], v, acc[hr]);
             if (++r == g.ring) r = 0;
         }
     }
 #pragma unroll
-    for (int hr = 0; hr < R; hr++) part[(w * R + hr) * 32 + lane] = acc[hr];
+    for (int hr = 0; hr < RB; hr++) part[(w * RB + hr) * 32 + lane] = acc[hr];
     __syncthreads();
-    for (int idx = threadIdx.x; idx < R * 32; idx += 512) {
-        const int hr = idx >> 5, l = idx & 31;
-        float sum = 0.0f;
+    for (int hr = w; hr < RB; hr += WV_WARPS) {
+        float a = 0.0f;
 #pragma unroll
-        for (int ww = 0; ww < 16; ww++) sum += part[(ww * R + hr) * 32 + l];
-        const int col = blockIdx.y * 32 + l;
-        if (col < g.dv) out[((int64_t)t * g.H + kvh * R + hr) * g.dv + col] = sum;
+        for (int ww = 0; ww < WV_WARPS; ww++) a += part[(ww * RB + hr) * 32 + lane];
+        acc_sm[hr * 32 + lane] = a;
     }
+    cluster.sync();
+    for (int hr = (int)blockIdx.z + WV_SPLIT * w; hr < nh; hr += WV_SPLIT * WV_WARPS) {
+        const int h = kvh * g.R + h0 + hr;
+        const float sk = sink ? sink[h] : -INFINITY;
+        float mx = sk;
+#pragma unroll
+        for (int z = 0; z < WV_SPLIT; z++) mx = fmaxf(mx, cluster.map_shared_rank(top, z)[hr]);
+        float tot = sink ? expf(sk - mx) : 0.0f, a = 0.0f;
+#pragma unroll
+        for (int z = 0; z < WV_SPLIT; z++) {
+            const float f = expf(cluster.map_shared_rank(top, z)[hr] - mx);                  // an empty slice: exp(-inf) = 0
+            tot = fmaf(f, cluster.map_shared_rank(sum, z)[hr], tot);
+            a = fmaf(f, cluster.map_shared_rank(acc_sm, z)[hr * 32 + lane], a);
+        }
+        const int col = blockIdx.y * 32 + lane;
+        if (col < g.dv) out[((int64_t)t * g.H + h) * g.dv + col] = a / tot;
+    }
+    cluster.sync();                                           // nobody leaves while its shared memory may still be read
 }
-template <int R>
-static cudaError_t wa_launch_group(cc_device* dev, const float* S, const float* v, float* out, const WaGeom& g, const float* sink, size_t smem) {
-    if (smem > 48 * 1024) { cudaError_t e = cudaFuncSetAttribute(wa_values_group_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); if (e != cudaSuccess) return e; }
-    wa_values_group_kernel<R><<<dim3((unsigned)(g.T * g.G), (unsigned)((g.dv + 31) / 32)), 512, smem, dev->stream>>>(S, v, out, g, sink);
+static size_t wa_slices_smem(int RB, int64_t maxn, int* slice_cap) {
+    *slice_cap = (int)((maxn + WV_SPLIT - 1) / WV_SPLIT);
+    return ((size_t)RB * *slice_cap + (size_t)WV_WARPS * RB * 32) * 4;
+}
+template <int RB>
+static cudaError_t wa_launch_slices(cc_device* dev, const float* S, const float* v, float* out, const WaGeom& g, const float* sink, size_t smem, int slice_cap) {
+    if (smem > 40 * 1024) { cudaError_t e = cudaFuncSetAttribute(wa_values_slices_kernel<RB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); if (e != cudaSuccess) return e; }
+    wa_values_slices_kernel<RB><<<dim3((unsigned)(g.T * g.G * ((g.R + RB - 1) / RB)), (unsigned)((g.dv + 31) / 32), WV_SPLIT), WV_THREADS, smem, dev->stream>>>(S, v, out, g, sink, slice_cap);
     return cudaSuccess;
 }
 // grid (dv tiles, query tiles, G)
@@ -1011,30 +1010,39 @@ __global__ void __launch_bounds__(WA_THREADS) wa_values_kernel(const float* __re
         for (int b = 0; b < 4; b++) acc[a][b] = 0.0f;
     // the next block of 16 keys (probabilities and values) is fetched into registers while the current one is multiplied: the loads' latency
     // hides behind the arithmetic of a CTA that often has its SM to itself
+    // keys are counted from the band's first one; a thread's rows, its column and its keys inside a block of 16 stay the same
     float pp[4], pv[4];
-    auto fetch = [&](int64_t j0) {
+    const float *Sp[4], *vp[4];
+    int p_lo[4], p_hi[4], vrow[4];
+    const int last_rel = (int)(i_last - band_lo);
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        const int idx = threadIdx.x + e * WA_THREADS;
+        {   // probabilities: consecutive threads read consecutive keys of one row
+            const int r = idx >> 4, tq = r / g.R, hr = r - tq * g.R;
+            const int64_t i = i_first + tq, lo = wa_lo(g, i);
+            const bool on = tq < tq_n;
+            p_lo[e] = (int)(lo - band_lo); p_hi[e] = on ? (int)(i - band_lo) : -1;
+            Sp[e] = on ? S + ((int64_t)(t0 + tq) * g.H + kvh * g.R + hr) * g.cap - p_lo[e] : S;
+        }
+        {   // values: consecutive threads read consecutive columns of one key
+            const int kk = idx >> 6, c = c0 + (idx & 63);
+            vrow[e] = (int)((band_lo + kk) % g.ring);
+            vp[e] = c < g.dv ? vring + kvh * g.vhs + c : nullptr;
+        }
+    }
+    auto fetch = [&](int j_rel) {                                // called with 0, 16, 32, ...
+        const int jp = j_rel + (threadIdx.x & 15);
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-            const int idx = threadIdx.x + e * WA_THREADS;
-            {   // probabilities: consecutive threads read consecutive keys of one row
-                const int r = idx >> 4, kk = idx & 15;
-                const int tq = r / g.R, hr = r - tq * g.R;
-                float p = 0.0f;
-                if (tq < tq_n) {
-                    const int64_t i = i_first + tq, lo = wa_lo(g, i), j = j0 + kk;
-                    if (j >= lo && j <= i) p = S[((int64_t)(t0 + tq) * g.H + kvh * g.R + hr) * g.cap + (j - lo)];
-                }
-                pp[e] = p;
-            }
-            {   // values: consecutive threads read consecutive columns of one key
-                const int kk = idx >> 6, c = idx & 63;
-                const int64_t j = j0 + kk;
-                pv[e] = (j <= i_last && c0 + c < g.dv) ? vring[(j % g.ring) * g.vrs + kvh * g.vhs + c0 + c] : 0.0f;
-            }
+            pp[e] = (jp >= p_lo[e] && jp <= p_hi[e]) ? Sp[e][jp] : 0.0f;
+            pv[e] = (vp[e] && j_rel + ((threadIdx.x + e * WA_THREADS) >> 6) <= last_rel) ? vp[e][(int64_t)vrow[e] * g.vrs] : 0.0f;
+            vrow[e] += WA_K;
+            while (vrow[e] >= g.ring) vrow[e] -= g.ring;
         }
     };
-    fetch(band_lo);
-    for (int64_t j0 = band_lo; j0 <= i_last; j0 += WA_K) {
+    fetch(0);
+    for (int j0 = 0; j0 <= last_rel; j0 += WA_K) {
 #pragma unroll
         for (int e = 0; e < 4; e++) {
             const int idx = threadIdx.x + e * WA_THREADS;
@@ -1042,7 +1050,7 @@ __global__ void __launch_bounds__(WA_THREADS) wa_values_kernel(const float* __re
             sv[idx >> 6][idx & 63] = pv[e];
         }
         __syncthreads();
-        if (j0 + WA_K <= i_last) fetch(j0 + WA_K);
+        if (j0 + WA_K <= last_rel) fetch(j0 + WA_K);
 #pragma unroll
         for (int kk = 0; kk < WA_K; kk++) {
             const float4 pv4 = *(const float4*)&sp[kk][ty * 4];
@@ -1120,34 +1128,32 @@ static int masked_attention_impl(cc_device* dev, const cc_view* q, const cc_view
     const int64_t band = reach - 1 + g.QT;                                             // keys a query tile can see
     const int64_t band_max = band < last + 1 ? band : last + 1;
     const bool few_rows = T * H <= 64;
-    if (few_rows && (size_t)R * dk * 4 <= 160 * 1024) {
-        const size_t smem = (size_t)R * dk * 4;
+    const int s_heads = R < WS_HEADS ? R : WS_HEADS;
+    if (few_rows && (size_t)s_heads * dk * 4 <= 160 * 1024) {
+        const size_t smem = (size_t)s_heads * dk * 4;
         if (smem > 48 * 1024) { cudaError_t e = cudaFuncSetAttribute(wa_scores_row_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); if (e != cudaSuccess) { cc_pool_free(dev, Sp, cls); return cc_fail(dev, CC_ERR_CUDA, "window_attention: %s", cudaGetErrorString(e)); } }
-        wa_scores_row_kernel<<<dim3((unsigned)((maxn + 7) / 8), (unsigned)T, (unsigned)G), 256, smem, dev->stream>>>(qp, fptr(kring), (float*)Sp, g, scale, r1 ? fptr(r1) : nullptr,
+        wa_scores_row_kernel<<<dim3((unsigned)((maxn + 15) / 16), (unsigned)T, (unsigned)(G * ((R + WS_HEADS - 1) / WS_HEADS))), 256, smem, dev->stream>>>(qp, fptr(kring), (float*)Sp, g, scale, r1 ? fptr(r1) : nullptr,
                                                                                                                       r2 ? fptr(r2) : nullptr);
     } else {
         dim3 g1((unsigned)((band_max + WA_TILE - 1) / WA_TILE), (unsigned)q_tiles, (unsigned)G);
         wa_scores_kernel<<<g1, WA_THREADS, 0, dev->stream>>>(qp, fptr(kring), (float*)Sp, g, scale, r1 ? fptr(r1) : nullptr, r2 ? fptr(r2) : nullptr);
     }
     dev->launches++;
-    const size_t group_smem = ((size_t)R * maxn + 16 * (size_t)R * 32) * 4;
-    const bool group_values = few_rows && (R == 2 || R == 4 || R == 8 || R == 16) && group_smem <= 160 * 1024;
-    const bool row_values = group_values || (few_rows && (size_t)maxn * 4 <= 160 * 1024);
+    const int RB = R >= 8 ? 8 : R >= 3 ? 4 : R;              // query heads a cluster of the few-row value kernel takes together
+    int slice_cap = 0;
+    const size_t slices_smem = wa_slices_smem(RB, maxn, &slice_cap);
+    const bool row_values = few_rows && slices_smem <= 160 * 1024;
     if (!row_values) {
         wa_softmax_kernel<<<(unsigned)((T * H + 7) / 8), 256, 0, dev->stream>>>((float*)Sp, g, sink ? fptr(sink) : nullptr);
         dev->launches++;
     }
-    if (group_values) {
+    if (row_values) {
         const float* sp = sink ? fptr(sink) : nullptr;
-        cudaError_t e = R == 2 ? wa_launch_group<2>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, group_smem)
-                      : R == 4 ? wa_launch_group<4>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, group_smem)
-                      : R == 8 ? wa_launch_group<8>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, group_smem)
-                               : wa_launch_group<16>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, group_smem);
+        cudaError_t e = RB == 8 ? wa_launch_slices<8>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, slices_smem, slice_cap)
+                      : RB == 4 ? wa_launch_slices<4>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, slices_smem, slice_cap)
+                      : RB == 2 ? wa_launch_slices<2>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, slices_smem, slice_cap)
+                                : wa_launch_slices<1>(dev, (const float*)Sp, vptr, (float*)o->base, g, sp, slices_smem, slice_cap);
         if (e != cudaSuccess) { cc_pool_free(dev, Sp, cls); return cc_fail(dev, CC_ERR_CUDA, "window_attention: %s", cudaGetErrorString(e)); }
-    } else if (row_values) {
-        const size_t smem = (size_t)maxn * 4;
-        if (smem > 48 * 1024) { cudaError_t e = cudaFuncSetAttribute(wa_values_row_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); if (e != cudaSuccess) { cc_pool_free(dev, Sp, cls); return cc_fail(dev, CC_ERR_CUDA, "window_attention: %s", cudaGetErrorString(e)); } }
-        wa_values_row_kernel<<<dim3((unsigned)(T * H), (unsigned)((dv + 31) / 32)), 128, smem, dev->stream>>>((const float*)Sp, vptr, (float*)o->base, g, sink ? fptr(sink) : nullptr);
     } else {
         dim3 g3((unsigned)((dv + WA_TILE - 1) / WA_TILE), (unsigned)q_tiles, (unsigned)G);
         wa_values_kernel<<<g3, WA_THREADS, 0, dev->stream>>>((const float*)Sp, vptr, (float*)o->base, g);
@@ -1365,7 +1371,7 @@ struct QkPrepArgs {
     int64_t pos0;
 };
 #define QKP_THREADS 256
-// one CTA per token.  First the inverse root mean squares -- one per head (a warp per head: lane-strided sum, butterfly) or one per projection
+// grid (tokens, blocks of heads); a norm over the whole projection takes one block.  First the inverse root mean squares -- one per head (a warp per head: lane-strided sum, butterfly) or one per projection
 // (thread-strided sums, butterfly, the warps' sums in warp order) -- then every element once: a rotated pair by the thread of its first
 // column, which reads both raw values and writes both results; all raw values were read for the sums before the barrier, so q may be
 // overwritten in place.
@@ -1374,12 +1380,13 @@ __global__ void __launch_bounds__(QKP_THREADS) qk_prepare_kernel(QkPrepArgs a) {
     float* inv = qkp_sm;
     float* red = qkp_sm + a.H + a.G;
     const int t = blockIdx.x, lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+    const int units_all = a.H + a.G, per_block = (units_all + gridDim.y - 1) / gridDim.y;
+    const int u0 = min(units_all, (int)blockIdx.y * per_block), u1 = min(units_all, u0 + per_block);       // this CTA's heads: queries', then keys'
     const float* qr = a.q + t * a.qrs;
     const float* kr = a.k + t * a.krs;
     float* qo = a.qo + (int64_t)t * a.H * a.dk;
-    const int units = a.H + a.G;
     if (a.norm == CC_QK_NORM_HEAD) {
-        for (int u = w; u < units; u += QKP_THREADS / 32) {
+        for (int u = u0 + w; u < u1; u += QKP_THREADS / 32) {
             const float* src = u < a.H ? qr + u * a.dk : kr + (u - a.H) * a.dk;
             float ss = 0.0f;
             for (int c = lane; c < a.dk; c += 32) ss = fmaf(src[c], src[c], ss);
@@ -1403,13 +1410,13 @@ __global__ void __launch_bounds__(QKP_THREADS) qk_prepare_kernel(QkPrepArgs a) {
             for (int u = threadIdx.x; u < (side ? a.G : a.H); u += QKP_THREADS) inv[(side ? a.H : 0) + u] = v;
         }
     } else {
-        for (int u = threadIdx.x; u < units; u += QKP_THREADS) inv[u] = 1.0f;
+        for (int u = u0 + threadIdx.x; u < u1; u += QKP_THREADS) inv[u] = 1.0f;
     }
     __syncthreads();
     const int64_t row = (a.pos0 + t) % a.ring;
     const float pos = (float)(a.pos0 + t);
-    for (int idx = threadIdx.x; idx < units * a.dk; idx += QKP_THREADS) {
-        const int u = idx / a.dk, c = idx - u * a.dk;
+    for (int idx = threadIdx.x; idx < (u1 - u0) * a.dk; idx += QKP_THREADS) {
+        const int ub = idx / a.dk, c = idx - ub * a.dk, u = u0 + ub;
         const bool is_q = u < a.H;
         const int ul = is_q ? u : u - a.H;
         const float* src = is_q ? qr + u * a.dk : kr + ul * a.dk;
@@ -1437,7 +1444,7 @@ __global__ void __launch_bounds__(QKP_THREADS) qk_prepare_kernel(QkPrepArgs a) {
     }
     const float* vr = a.v + t * a.vrs;
     float* vd = a.vring + row * a.G * a.dv;
-    for (int c = threadIdx.x; c < a.G * a.dv; c += QKP_THREADS) vd[c] = vr[c];
+    for (int c = blockIdx.y * QKP_THREADS + threadIdx.x; c < a.G * a.dv; c += gridDim.y * QKP_THREADS) vd[c] = vr[c];
 }
 static int qk_prepare_impl(cc_device* dev, QkPrepArgs a, int64_t T, const cc_view* kring, const cc_view* vring, int32_t qk_norm, const cc_view* q_w, const cc_view* k_w, float eps,
                            const cc_view* freq, int32_t pairing, int32_t offset, float mag, int64_t pos0, int32_t H, int32_t G, int32_t dk, int32_t dv) {
@@ -1462,7 +1469,8 @@ static int qk_prepare_impl(cc_device* dev, QkPrepArgs a, int64_t T, const cc_vie
     a.step = pairing == CC_ROPE_HALVES ? 1 : 2; a.gap = pairing == CC_ROPE_HALVES ? (int)half : 1; a.eps = eps; a.mag = mag; a.pos0 = pos0;
     const size_t smem = (size_t)(H + G + QKP_THREADS / 32) * 4;
     CC_REQUIRE(dev, smem <= 48 * 1024, "qk_prepare_append: too many heads");
-    qk_prepare_kernel<<<(unsigned)T, QKP_THREADS, smem, dev->stream>>>(a);
+    const int blocks = qk_norm == CC_QK_NORM_ROW ? 1 : (H + G + QKP_THREADS / 32 - 1) / (QKP_THREADS / 32);       // a warp per head
+    qk_prepare_kernel<<<dim3((unsigned)T, (unsigned)blocks), QKP_THREADS, smem, dev->stream>>>(a);
     CC_LAUNCH_CHECK(dev);
     return CC_OK;
 }
