@@ -1523,9 +1523,11 @@ __device__ __forceinline__ void latent_append_row(const LatAppend& a, int t, int
     const float eps = a.eps, mag = a.mag;
     float* dst = a.ring + ((pos0 + t) % a.ring_rows) * cols;
     float ss = 0.0f;
+#pragma unroll 8
     for (int c = lane; c < rank; c += 32) ss = fmaf(src[c], src[c], ss);
     ss = warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
+#pragma unroll 8
     for (int c = lane; c < rank; c += 32) dst[c] = src[c] * inv * (nw ? nw[c] : 1.0f);
     for (int i = lane; i < half; i += 32) {
         float ou, ov;
