@@ -1568,7 +1568,7 @@ struct HpArgs {
     const float *freq, *gate;     // gate (rest == 0 only): output (t, h, v) is multiplied by sigmoid(gate[t * grs + h * ghs + v * gvs]); NULL: not gated
     int T, H, n_in, rest, n_out, half, step, gap, ghs, gvs;
     float mag;
-    LatAppend app;                // app.ring != NULL: the grid has one more z plane, whose CTAs of head 0 write the tokens' cache rows
+    LatAppend app;                // app.ring != NULL: the grid has one more z plane, the first, whose CTAs of head 0 write the tokens' cache rows
 };
 // grid (ceil(T / 8), H, ceil(n_out / 4)): the CTA stages 8 tokens' x[t, h, :n_in]; a warp owns one output coordinate for those tokens:
 // lane-strided partial sums over n_in, then the butterfly -- one order per output, whatever T is.  W: [H * n_out, n_in], rows read
@@ -1576,7 +1576,8 @@ struct HpArgs {
 __global__ void __launch_bounds__(128) head_project_kernel(HpArgs a) {
     extern __shared__ float hp_sm[];
     const int t0 = blockIdx.x * HP_TOK, h = blockIdx.y, T = a.T, H = a.H, n_in = a.n_in, rest = a.rest, n_out = a.n_out, half = a.half;
-    if (a.app.ring && blockIdx.z == gridDim.z - 1) {
+    const int z = (int)blockIdx.z - (a.app.ring ? 1 : 0);
+    if (z < 0) {
         if (h == 0)
             for (int tt = threadIdx.x >> 5; tt < HP_TOK && t0 + tt < T; tt += 4) latent_append_row(a.app, t0 + tt, threadIdx.x & 31);
         return;
@@ -1586,7 +1587,7 @@ __global__ void __launch_bounds__(128) head_project_kernel(HpArgs a) {
         const int tt = i / n_in, d = i - tt * n_in;
         hp_sm[i] = t0 + tt < T ? a.x[(t0 + tt) * a.xrs + h * xs + d] : 0.0f;
     }
-    if (blockIdx.z == 0) {
+    if (z == 0) {
         // the carried columns: the first 2 * half of them are rotated on the way when a frequency table is given
         for (int i = threadIdx.x; i < HP_TOK * half; i += 128) {
             const int tt = i / half, p = i - tt * half;
@@ -1602,7 +1603,7 @@ __global__ void __launch_bounds__(128) head_project_kernel(HpArgs a) {
         }
     }
     __syncthreads();
-    const int v = blockIdx.z * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int v = z * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (v >= n_out) return;
     const float* wp = a.W + ((int64_t)h * n_out + v) * n_in;
     float acc[HP_TOK];
