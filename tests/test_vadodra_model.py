@@ -220,7 +220,7 @@ CONFIGS = {
     "mixers_only": config([window(mlp=None), latent(mlp=None), window(size=11, mlp=None)], embed_scale=0.25),
     "heads_that_do_not_fill_a_tile": config([window(heads=33, kv_heads=1, dim=4, rot=2), window(heads=21, kv_heads=7, dim=6, rot=2, size=30)], width=40, vocab=33),
     "many_heads": config([latent(heads=70, dim=2, rot_dim=2, vdim=2, kv_rank=5, mlp=None), latent(heads=33, dim=2, rot_dim=2, vdim=3, kv_rank=5, kv_from=0)], width=40, vocab=33),
-    "aligned_for_tensor_cores": config([latent(heads=4, dim=32, rot_dim=16, vdim=32, kv_rank=64, mlp=dense(192, 1.1)), window(heads=4, kv_heads=2, dim=32, size=40, rot=16, mlp=dense(320)),
+    "aligned_for_tensor_cores": config([latent(heads=4, dim=32, rot_dim=16, vdim=32, kv_rank=64, mlp=dense(192, 1.1)), window(heads=6, kv_heads=2, dim=32, size=45, rot=16, mlp=dense(320)),
                                         latent(heads=2, dim=64, rot_dim=16, vdim=64, kv_rank=64, kv_from=0, mlp=dense(128)), window(heads=2, kv_heads=1, dim=64, size=100, rot=64, mlp=None)],
                                        width=128, vocab=256),
     "wide_rows": config([latent(heads=2, dim=16, rot_dim=8, vdim=24, kv_rank=40), window(heads=10, kv_heads=5, dim=48, size=50, rot=48, mlp=dense(700, 3.0))], width=1064, vocab=64),
